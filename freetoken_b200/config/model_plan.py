@@ -75,11 +75,13 @@ class RunEntry:
     ``layer`` indexes :attr:`ModelPlan.layers` (a layer named by two stops runs
     twice with the same weights).  Every stop has a cache of its own unless
     ``reads_cache_of`` names an earlier stop of the schedule: then the stop
-    writes nothing and its mixer reads what that stop wrote.
+    writes nothing and its mixer reads what that stop wrote.  ``stream_map`` indexes
+    :attr:`ModelPlan.stream_maps`: what happens to the residual stream right before the stop.
     """
 
     layer: int
     reads_cache_of: Optional[int] = None
+    stream_map: Optional[int] = None
 
     @property
     def owns_cache(self) -> bool:
@@ -101,6 +103,8 @@ class ModelPlan:
     max_position: int
     # residual streams per token (hyper-connections); 1: the plain residual stream [T, H]
     residual_streams: int = 1
+    # maps of the (plain) residual stream that stops of the schedule may name
+    stream_maps: Tuple[PartSpec, ...] = ()
 
     def validate(self) -> None:
         n = len(self.layers)
@@ -111,6 +115,13 @@ class ModelPlan:
         for i, stop in enumerate(self.schedule):
             if not 0 <= stop.layer < n:
                 raise ValueError(f"schedule[{i}] names layer {stop.layer}, outside 0..{n - 1}")
+            if stop.stream_map is not None:
+                if not 0 <= stop.stream_map < len(self.stream_maps):
+                    raise ValueError(f"schedule[{i}] names stream map {stop.stream_map}, the plan has "
+                                     f"{len(self.stream_maps)}")
+                if self.residual_streams != 1:
+                    raise ValueError(f"schedule[{i}]: a stream map works on the plain residual stream, the plan "
+                                     f"has {self.residual_streams} streams")
             src = stop.reads_cache_of
             if src is None:
                 continue

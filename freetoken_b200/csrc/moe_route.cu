@@ -206,7 +206,7 @@ __global__ void __launch_bounds__(SMALL_WARPS * 32) route_small_kernel(
     const float* __restrict__ logits, const float* __restrict__ bias, int* __restrict__ ids,
     float* __restrict__ weights, int* __restrict__ counts, int* __restrict__ offsets,
     int* __restrict__ sorted_route, int* __restrict__ sorted_token, int* __restrict__ active, int T, int E,
-    int k, int softmax_scoring, int renormalize, float scale, int terms, int groups, int keep) {
+    int busy_of, int k, int softmax_scoring, int renormalize, float scale, int terms, int groups, int keep) {
   extern __shared__ float smem[];  // [T][2][E] scores and choices, then ints: ids [T*k], counts [E], before [E]
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int R = T * k;
@@ -239,7 +239,7 @@ __global__ void __launch_bounds__(SMALL_WARPS * 32) route_small_kernel(
     // exclusive scan over the experts: a lane takes a run of consecutive experts
     const int per = (E + 31) / 32, begin = lane * per, end = min(E, begin + per);
     int rows = 0, busy = 0;
-    for (int e = begin; e < end; ++e) { rows += s_cnt[e]; busy += s_cnt[e] > 0; }
+    for (int e = begin; e < end; ++e) { rows += s_cnt[e]; busy += s_cnt[e] > 0 && e < busy_of; }
     int rows_before = rows, busy_before = busy;
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
@@ -253,12 +253,12 @@ __global__ void __launch_bounds__(SMALL_WARPS * 32) route_small_kernel(
     for (int e = begin; e < end; ++e) {
       s_before[e] = rows_before;
       offsets[e] = rows_before;
-      if (s_cnt[e] > 0) active[busy_before++] = e;
+      if (s_cnt[e] > 0 && e < busy_of) active[busy_before++] = e;
       rows_before += s_cnt[e];
     }
     if (lane == 0) {
       offsets[E] = total_rows;
-      active[E] = total_busy;
+      active[busy_of] = total_busy;
     }
   }
   __syncthreads();
@@ -369,11 +369,11 @@ __global__ void moe_count_kernel(const int* __restrict__ ids, int* __restrict__ 
 
 // offsets[e] = sum counts[<e]; sorted_route[offsets[e] + i] = i-th route of
 // expert e in ascending route order; sorted_token = sorted_route / k;
-// active[j] = j-th expert that has routes (ascending), active[E] = how many.
+// active[j] = j-th expert below busy_of that has routes (ascending), active[busy_of] = how many.
 __global__ void moe_scatter_kernel(const int* __restrict__ ids, const int* __restrict__ counts,
                                    int* __restrict__ offsets, int* __restrict__ sorted_route,
                                    int* __restrict__ sorted_token, int* __restrict__ active,
-                                   int R, int E, int k) {
+                                   int R, int E, int busy_of, int k) {
   const int lane = threadIdx.x & 31;
   pdl_wait();
 
@@ -394,11 +394,9 @@ __global__ void moe_scatter_kernel(const int* __restrict__ ids, const int* __res
   if (lane == 0) {
     const int mine = counts[e];
     offsets[e] = before;
-    if (mine > 0) active[busy_before] = e;
-    if (e == E - 1) {
-      offsets[E] = before + mine;
-      active[E] = busy_before + (mine > 0);
-    }
+    if (mine > 0 && e < busy_of) active[busy_before] = e;
+    if (e == E - 1) offsets[E] = before + mine;
+    if (e == busy_of - 1) active[busy_of] = busy_before + (mine > 0);
   }
   int at = before;
   for (int base = 0; base < R; base += 32 * SCAN) {
@@ -454,7 +452,8 @@ __global__ void __launch_bounds__(SORT_CHUNK) moe_chunk_count_kernel(const int* 
 // carry for the offsets and for the number of busy experts.
 __global__ void __launch_bounds__(1024) moe_chunk_scan_kernel(int* __restrict__ chunk_counts,
                                                               int* __restrict__ counts, int* __restrict__ offsets,
-                                                              int* __restrict__ active, int chunks, int E) {
+                                                              int* __restrict__ active, int chunks, int E,
+                                                              int busy_of) {
   __shared__ int scan_rows[1024], scan_busy[1024];
   __shared__ int carry_rows, carry_busy;
   if (threadIdx.x == 0) { carry_rows = 0; carry_busy = 0; }
@@ -478,7 +477,7 @@ __global__ void __launch_bounds__(1024) moe_chunk_scan_kernel(int* __restrict__ 
       counts[e] = total;
     }
     scan_rows[threadIdx.x] = total;
-    scan_busy[threadIdx.x] = total > 0;
+    scan_busy[threadIdx.x] = total > 0 && e < busy_of;
     __syncthreads();
     for (int o = 1; o < (int)blockDim.x; o <<= 1) {
       const int a = threadIdx.x >= (unsigned)o ? scan_rows[threadIdx.x - o] : 0;
@@ -491,11 +490,9 @@ __global__ void __launch_bounds__(1024) moe_chunk_scan_kernel(int* __restrict__ 
     if (e < E) {
       const int before = carry_rows + scan_rows[threadIdx.x] - total;
       offsets[e] = before;
-      if (total > 0) active[carry_busy + scan_busy[threadIdx.x] - 1] = e;
-      if (e == E - 1) {
-        offsets[E] = before + total;
-        active[E] = carry_busy + scan_busy[threadIdx.x];
-      }
+      if (total > 0 && e < busy_of) active[carry_busy + scan_busy[threadIdx.x] - 1] = e;
+      if (e == E - 1) offsets[E] = before + total;
+      if (e == busy_of - 1) active[busy_of] = carry_busy + scan_busy[threadIdx.x];
     }
     __syncthreads();
     if (threadIdx.x == blockDim.x - 1) {
@@ -562,13 +559,13 @@ int ft_router_select(const float* logits, const float* bias, int* ids, float* we
   return FT_OK;
 }
 
-// router_select + moe_sort in one launch; T <= 8 tokens, k <= 32.
+// router_select + moe_sort in one launch; T <= 8 tokens, k <= 32.  `busy_of` as in ft_moe_sort.
 int ft_route_small(const float* logits, const float* bias, int* ids, float* weights, int* counts,
-                   int* offsets, int* sorted_route, int* sorted_token, int* active, int T, int E, int k,
+                   int* offsets, int* sorted_route, int* sorted_token, int* active, int T, int E, int busy_of, int k,
                    int softmax_scoring, int renormalize, float scale, int terms, int groups, int keep,
                    cudaStream_t stream) {
   if (T <= 0) return FT_OK;
-  if (T > SMALL_WARPS || k <= 0 || k > 32 || k > E || terms < 1) return FT_ERR_SHAPE;
+  if (T > SMALL_WARPS || k <= 0 || k > 32 || k > E || terms < 1 || busy_of < 1 || busy_of > E) return FT_ERR_SHAPE;
   if (groups < 1 || groups > 256 || E % groups || keep < 1 || keep > groups || keep * (E / groups) < k)
     return FT_ERR_SHAPE;
   const size_t smem = (size_t)T * 2 * E * sizeof(float) + ((size_t)T * k + 2 * (size_t)E) * sizeof(int);
@@ -576,7 +573,7 @@ int ft_route_small(const float* logits, const float* bias, int* ids, float* weig
   if (smem > 48 * 1024)
     cudaFuncSetAttribute(route_small_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   launch_pdl(route_small_kernel, dim3(1), dim3(SMALL_WARPS * 32), smem, stream, logits, bias, ids, weights,
-             counts, offsets, sorted_route, sorted_token, active, T, E, k, softmax_scoring, renormalize, scale,
+             counts, offsets, sorted_route, sorted_token, active, T, E, busy_of, k, softmax_scoring, renormalize, scale,
              terms, groups, keep);
   FT_LAUNCH_CHECK();
   return FT_OK;
@@ -599,10 +596,13 @@ long long ft_moe_sort_scratch(int R, int E) {
 }
 
 // `scratch` (ft_moe_sort_scratch ints) selects the chunked sort; without it one
-// warp per expert walks the routes (few routes: a decode batch).
+// warp per expert walks the routes (few routes: a decode batch).  Only ids below `busy_of` enter the
+// list of busy experts (active[0 ..], their number at active[busy_of]): the ids from there on name
+// no expert with weights; their routes lie behind all others.
 int ft_moe_sort(const int* ids, int* counts, int* offsets, int* sorted_route, int* sorted_token,
-                int* active, int* scratch, int R, int E, int k, cudaStream_t stream) {
+                int* active, int* scratch, int R, int E, int busy_of, int k, cudaStream_t stream) {
   if (R <= 0) return FT_OK;
+  if (busy_of < 1 || busy_of > E) return FT_ERR_SHAPE;
   if (scratch) {
     const int chunks = (R + SORT_CHUNK - 1) / SORT_CHUNK;
     const size_t hist = (size_t)E * sizeof(int), cur = 4 * hist;
@@ -613,7 +613,7 @@ int ft_moe_sort(const int* ids, int* counts, int* offsets, int* sorted_route, in
     }
     moe_chunk_count_kernel<<<chunks, SORT_CHUNK, hist, stream>>>(ids, scratch, R, E);
     moe_chunk_scan_kernel<<<1, E < 1024 ? ((E + 31) / 32) * 32 : 1024, 0, stream>>>(scratch, counts, offsets,
-                                                                                   active, chunks, E);
+                                                                                   active, chunks, E, busy_of);
     moe_chunk_scatter_kernel<<<(chunks + 3) / 4, 128, cur, stream>>>(ids, scratch, offsets, sorted_route,
                                                                      sorted_token, R, E, k, chunks);
     FT_LAUNCH_CHECK();
@@ -623,7 +623,7 @@ int ft_moe_sort(const int* ids, int* counts, int* offsets, int* sorted_route, in
   const int blocks = (E + warps - 1) / warps;
   launch_pdl(moe_count_kernel, dim3(blocks), dim3(warps * 32), 0, stream, ids, counts, R, E);
   launch_pdl(moe_scatter_kernel, dim3(blocks), dim3(warps * 32), 0, stream, ids, (const int*)counts, offsets,
-             sorted_route, sorted_token, active, R, E, k);
+             sorted_route, sorted_token, active, R, E, busy_of, k);
   FT_LAUNCH_CHECK();
   return FT_OK;
 }

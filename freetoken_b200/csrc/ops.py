@@ -350,33 +350,102 @@ def softcap(x: torch.Tensor, cap: float) -> None:
 
 
 # ------------------------------------- sandwich norms, sums of mixers, biases, gated rows
-def norm_add(branch: torch.Tensor, residual: torch.Tensor, weight: torch.Tensor, eps: float,
+class RoutedRows:
+    """What a routed feed-forward hands on, not added up yet: ``rows`` ``[T, k, H]``, of which slots
+    whose id (``ids`` ``[T, k]``) is ``experts`` or more were never written - such a slot hands the
+    branch's input ``source`` (``[T, H]``) back, times its weight (``weights`` ``[T, k]``) -, and ``extra``
+    (``[T, H]`` or None), one more row per token.  The value of a token is the sum of all that."""
+
+    __slots__ = ("rows", "ids", "weights", "experts", "source", "extra")
+
+    def __init__(self, rows, ids=None, weights=None, experts: int = 0, source=None, extra=None):
+        self.rows, self.ids, self.weights, self.experts = rows, ids, weights, int(experts)
+        self.source, self.extra = source, extra
+
+
+def _branch_args(branch, T: int, H: int, name: str):
+    """``(rows tensor, k, ids, weights, experts, source, extra)`` of a branch output, checked."""
+    if not isinstance(branch, RoutedRows):
+        branch = RoutedRows(branch)
+    rows = branch.rows
+    _need(rows, "branch")
+    k = rows.shape[1] if rows.dim() == 3 else 1
+    if rows.shape[0] != T or rows.shape[-1] != H:
+        raise KernelError(f"{name}: shapes do not match")
+    if branch.ids is not None:
+        _need(branch.ids, "ids", torch.int32)
+        _need(branch.weights, "weights", torch.float32)
+        _need(branch.source, "source", rows.dtype)
+        if branch.ids.numel() != T * k or branch.weights.numel() != T * k or branch.source.shape != (T, H):
+            raise KernelError(f"{name}: one id and one weight per partial row, one source row per token")
+    if branch.extra is not None:
+        _need(branch.extra, "extra", rows.dtype)
+        if branch.extra.shape != (T, H):
+            raise KernelError(f"{name}: one extra row per token")
+    return rows, k, branch.ids, branch.weights, branch.experts, branch.source, branch.extra
+
+
+def norm_add(branch, residual: torch.Tensor, weight: torch.Tensor, eps: float,
              plus_one: bool, mult: float, part_scale: Optional[torch.Tensor] = None,
              next_weight: Optional[torch.Tensor] = None, next_eps: float = 0.0,
-             next_plus_one: bool = False, next_out: Optional[torch.Tensor] = None) -> None:
+             next_plus_one: bool = False, next_out: Optional[torch.Tensor] = None,
+             copy_out: Optional[torch.Tensor] = None) -> None:
     """residual += mult * rms(z) * (weight [+1]) with z = sum_j part_scale[j] * branch[:, j, :]
-    (``branch`` is ``[T, H]`` or ``[T, k, H]``; float32 throughout).  With ``next_weight`` the new
-    residual rows are RMS-normed once more into ``next_out``."""
-    _need(branch, "branch")
+    (``branch`` is ``[T, H]`` or ``[T, k, H]``, or :class:`RoutedRows`; float32 throughout).  With
+    ``next_weight`` the new residual rows are RMS-normed once more into ``next_out``; with ``copy_out``
+    (``[T, H]``, rows may lie further apart) they also leave as they are, in the activation type."""
     _need(residual, "residual", torch.float32)
     _need(weight, "weight", torch.float32)
     T, H = residual.shape
-    k = branch.shape[1] if branch.dim() == 3 else 1
-    if branch.shape[0] != T or branch.shape[-1] != H or weight.numel() != H:
+    rows, k, ids, weights, experts, source, extra = _branch_args(branch, T, H, "norm_add")
+    if weight.numel() != H:
         raise KernelError("norm_add: shapes do not match")
     if part_scale is not None:
         _need(part_scale, "part_scale", torch.float32)
-        if part_scale.numel() != k:
-            raise KernelError("norm_add: one scale per partial row")
+        if part_scale.numel() != k or ids is not None:
+            raise KernelError("norm_add: one scale per partial row (and no ids beside scales)")
     if next_weight is not None:
         _need(next_weight, "next_weight", torch.float32)
-        _need(next_out, "next_out", branch.dtype)
+        _need(next_out, "next_out", rows.dtype)
         if next_out.shape != residual.shape or next_weight.numel() != H:
             raise KernelError("norm_add: the second norm's shapes do not match")
-    f = _fn("rowwise", "ft_norm_add", "p i p p i f f p p i f p i i i")
-    _check(f(_ptr(branch), k, _ptr(part_scale), _ptr(weight), int(plus_one), float(eps), float(mult),
-             _ptr(residual), _ptr(next_weight), int(next_plus_one), float(next_eps), _ptr(next_out), T, H,
-             code(branch.dtype), _stream()), "norm_add")
+    if copy_out is not None:
+        _need(copy_out, "copy_out", rows.dtype, contiguous=False)
+        if copy_out.shape != residual.shape or copy_out.stride(1) != 1:
+            raise KernelError("norm_add: copy_out must be [T, H] with unit stride")
+    f = _fn("rowwise", "ft_norm_add", "p i p p p i p p p i f f p p i f p p q i i i")
+    _check(f(_ptr(rows), k, _ptr(part_scale), _ptr(ids), _ptr(weights), experts, _ptr(source), _ptr(extra),
+             _ptr(weight), int(plus_one), float(eps), float(mult), _ptr(residual), _ptr(next_weight),
+             int(next_plus_one), float(next_eps), _ptr(next_out), _ptr(copy_out),
+             copy_out.stride(0) if copy_out is not None else 0, T, H, code(rows.dtype), _stream()), "norm_add")
+
+
+def branch_sum(branch, out: torch.Tensor) -> None:
+    """out[t, :] = the value of token t of ``branch`` (``[T, k, H]`` or :class:`RoutedRows`), summed in float32."""
+    T, H = out.shape
+    rows, k, ids, weights, experts, source, extra = _branch_args(branch, T, H, "branch_sum")
+    _need(out, "out", rows.dtype)
+    f = _fn("rowwise", "ft_branch_sum", "p i p p i p p p i i i")
+    _check(f(_ptr(rows), k, _ptr(ids), _ptr(weights), experts, _ptr(source), _ptr(extra), _ptr(out), T, H,
+             code(rows.dtype), _stream()), "branch_sum")
+
+
+def cast_rows(x: torch.Tensor, dst: torch.Tensor, branch=None) -> None:
+    """dst[t, :] = x[t, :] (float32 rows into the activation type; ``dst`` rows may lie further apart).
+    With ``branch`` (as for :func:`branch_sum`) its value joins ``x`` in place first."""
+    _need(x, "x", torch.float32)
+    _need(dst, "dst", contiguous=False)
+    if dst.shape != x.shape or dst.dim() != 2 or dst.stride(1) != 1:
+        raise KernelError("cast_rows: dst must be [T, H] with unit stride")
+    T, H = x.shape
+    rows, k, ids, weights, experts, source, extra = (None, 0, None, None, 0, None, None)
+    if branch is not None:
+        rows, k, ids, weights, experts, source, extra = _branch_args(branch, T, H, "cast_rows")
+        if rows.dtype != dst.dtype:
+            raise KernelError("cast_rows: the branch and dst must have one element type")
+    f = _fn("rowwise", "ft_cast_rows", "p p i p p i p p p q i i i")
+    _check(f(_ptr(x), _ptr(rows), k, _ptr(ids), _ptr(weights), experts, _ptr(source), _ptr(extra), _ptr(dst),
+             dst.stride(0), T, H, code(dst.dtype), _stream()), "cast_rows")
 
 
 def scaled_sum(parts: torch.Tensor, scale: torch.Tensor, out: torch.Tensor) -> None:
@@ -1242,7 +1311,7 @@ def route_small(logits: torch.Tensor, bias: Optional[torch.Tensor], ids: torch.T
                 weights: torch.Tensor, counts: torch.Tensor, offsets: torch.Tensor,
                 sorted_route: torch.Tensor, sorted_token: torch.Tensor, active: torch.Tensor, k: int,
                 softmax_scoring: bool, renormalize: bool, scale: float, terms: int = 1, groups: int = 1,
-                keep: int = 1) -> None:
+                keep: int = 1, busy_of: int = 0) -> None:
     """:func:`router_select` and :func:`moe_sort` in one launch (same results)."""
     _need(logits, "logits", torch.float32)
     _need(weights, "weights", torch.float32)
@@ -1253,14 +1322,15 @@ def route_small(logits: torch.Tensor, bias: Optional[torch.Tensor], ids: torch.T
         _need(t, name, torch.int32)
     T, E = logits.shape[0], logits.shape[1] // terms
     R = T * k
-    if logits.shape[1] != E * terms or not route_small_takes(T, E, k):
+    busy_of = busy_of or E
+    if logits.shape[1] != E * terms or not route_small_takes(T, E, k) or not 1 <= busy_of <= E:
         raise KernelError(f"route_small: refuses {T} tokens, {E} experts, top-{k}")
     if counts.numel() < E or offsets.numel() < E + 1 or sorted_route.numel() < R \
-            or sorted_token.numel() < R or active.numel() < E + 1 or ids.numel() < R or weights.numel() < R:
+            or sorted_token.numel() < R or active.numel() < busy_of + 1 or ids.numel() < R or weights.numel() < R:
         raise KernelError("route_small: output buffers are too small")
-    f = _fn("moe_route", "ft_route_small", "p p p p p p p p p i i i i i f i i i")
+    f = _fn("moe_route", "ft_route_small", "p p p p p p p p p i i i i i i f i i i")
     _check(f(_ptr(logits), _ptr(bias), _ptr(ids), _ptr(weights), _ptr(counts), _ptr(offsets),
-             _ptr(sorted_route), _ptr(sorted_token), _ptr(active), T, E, k, int(softmax_scoring),
+             _ptr(sorted_route), _ptr(sorted_token), _ptr(active), T, E, busy_of, k, int(softmax_scoring),
              int(renormalize), float(scale), int(terms), int(groups), int(keep), _stream()), "route_small")
 
 
@@ -1285,9 +1355,11 @@ def router_logits(x: torch.Tensor, w: torch.Tensor, logits: torch.Tensor) -> Non
 
 def moe_sort(ids: torch.Tensor, counts: torch.Tensor, offsets: torch.Tensor,
              sorted_route: torch.Tensor, sorted_token: torch.Tensor, active: torch.Tensor,
-             num_experts: int, k: int, scratch: Optional[torch.Tensor] = None) -> None:
+             num_experts: int, k: int, scratch: Optional[torch.Tensor] = None, busy_of: int = 0) -> None:
     """Stable counting sort of the ``T*k`` routes by expert; ``active`` gets the
-    experts that have routes (ascending) and, at index ``num_experts``, their number.
+    experts that have routes (ascending) and, at index ``num_experts``, their number
+    (``busy_of``: only ids below it, their number at index ``busy_of`` - the ids from there on
+    stand for no expert with weights, and their routes lie behind all others).
     With ``scratch`` (int32, :func:`moe_sort_scratch` elements) the routes are
     sorted in chunks, which is faster from a few thousand routes on."""
     for name, t in (("ids", ids), ("counts", counts), ("offsets", offsets),
@@ -1295,17 +1367,18 @@ def moe_sort(ids: torch.Tensor, counts: torch.Tensor, offsets: torch.Tensor,
                     ("active", active)):
         _need(t, name, torch.int32)
     R = ids.numel()
-    if counts.numel() < num_experts or offsets.numel() < num_experts + 1 \
+    busy_of = busy_of or num_experts
+    if counts.numel() < num_experts or not 1 <= busy_of <= num_experts or offsets.numel() < num_experts + 1 \
             or sorted_route.numel() < R or sorted_token.numel() < R \
-            or active.numel() < num_experts + 1:
+            or active.numel() < busy_of + 1:
         raise KernelError("moe_sort: output buffers are too small")
     if scratch is not None:
         _need(scratch, "scratch", torch.int32)
         if scratch.numel() < moe_sort_scratch(R, num_experts):
             raise KernelError("moe_sort: the scratch buffer is too small")
-    f = _fn("moe_route", "ft_moe_sort", "p p p p p p p i i i")
+    f = _fn("moe_route", "ft_moe_sort", "p p p p p p p i i i i")
     _check(f(_ptr(ids), _ptr(counts), _ptr(offsets), _ptr(sorted_route), _ptr(sorted_token),
-             _ptr(active), _ptr(scratch), R, num_experts, k, _stream()), "moe_sort")
+             _ptr(active), _ptr(scratch), R, num_experts, busy_of, k, _stream()), "moe_sort")
     if scratch is not None:
         global LAUNCHES
         LAUNCHES += 1      # three kernels instead of two

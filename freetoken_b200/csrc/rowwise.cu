@@ -13,6 +13,8 @@
 //   gate_heads      o[t,h,:] *= sigmoid(z[t,h])
 //   activation      y = f(x): relu(x)^2, tanh-GELU, SiLU
 //   softcap         y = cap * tanh(y / cap)
+//   norm_add        x += mult * rms(z) * w, z a branch's rows summed; optionally the next norm and a copy
+//   branch_sum, cast_rows   z as one row; x += z and its copy in the activation type
 #include "common.cuh"
 
 namespace ft {
@@ -265,11 +267,23 @@ __global__ void __launch_bounds__(256) softcap_kernel(float* __restrict__ x, lon
   if (i < n) x[i] = cap * tanhf(x[i] / cap);
 }
 
-// ------------------------------------------------- a branch's own norm, then the residual
-// z = sum_j s_j * branch[t, j, :] (float32; s_j = 1 without scales); the residual takes
-// mult * rms(z) * (w [+1]).  With a second weight the new residual row is normed once more
-// in the same pass and leaves as the next sublayer's input.  A block owns a token; z, then the
-// new residual row, stay in shared memory between the passes.
+// ------------------------------------------------- what a feed-forward hands on, row by row
+// A branch output of a token is a sum of rows that nobody has added yet (float32, in this order):
+//   z = sum_j s_j * rows[t, j, :]      the k partial rows (s_j = 1 without scales)
+//     + extra[t, :]                     one more row per token (a shared expert), if there is one
+//     + c_t * source[t, :]              c_t = sum of weights[t, j] over the slots whose id is >= experts
+// With ids, slots whose id is >= `experts` have no row (it is never written, so it is not read): such
+// a slot hands the branch's own input back, times its weight.
+struct BranchArgs {
+  const void* rows;        // [T, k, H]
+  const float* part_scale; // [k] or nullptr
+  const int* ids;          // [T, k] or nullptr: every slot has a row
+  const float* weights;    // [T, k]
+  const void* source;      // [T, H]
+  const void* extra;       // [T, H] or nullptr
+  int k, experts;
+};
+
 __device__ __forceinline__ void store4f(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
 __device__ __forceinline__ void store4f(__nv_bfloat16* p, float4 v) {
   uint2 raw;
@@ -278,24 +292,128 @@ __device__ __forceinline__ void store4f(__nv_bfloat16* p, float4 v) {
   *reinterpret_cast<uint2*>(p) = raw;
 }
 
+// the value of column c, and of columns 4g .. 4g + 3, of token t's branch
+template <typename AT>
+__device__ __forceinline__ float branch_at(const BranchArgs& b, int t, int H, int c) {
+  const AT* rows = (const AT*)b.rows + (size_t)t * b.k * H + c;
+  float z = 0.f, back = 0.f;
+  for (int j = 0; j < b.k; ++j) {
+    if (b.ids && b.ids[(size_t)t * b.k + j] >= b.experts) {
+      back += b.weights[(size_t)t * b.k + j];
+      continue;
+    }
+    const float v = to_float(rows[(size_t)j * H]);
+    z = b.part_scale ? fmaf(b.part_scale[j], v, z) : z + v;
+  }
+  if (b.extra) z += to_float(((const AT*)b.extra)[(size_t)t * H + c]);
+  if (back != 0.f) z = fmaf(back, to_float(((const AT*)b.source)[(size_t)t * H + c]), z);
+  return z;
+}
+template <typename AT>
+__device__ __forceinline__ float4 branch_at4(const BranchArgs& b, int t, int H, int gi) {
+  const AT* rows = (const AT*)b.rows + (size_t)t * b.k * H + 4 * gi;
+  float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
+  float back = 0.f;
+  for (int j = 0; j < b.k; ++j) {
+    if (b.ids && b.ids[(size_t)t * b.k + j] >= b.experts) {
+      back += b.weights[(size_t)t * b.k + j];
+      continue;
+    }
+    const float4 v = load4f(rows + (size_t)j * H);
+    if (b.part_scale) {
+      const float s = b.part_scale[j];
+      z.x = fmaf(s, v.x, z.x); z.y = fmaf(s, v.y, z.y); z.z = fmaf(s, v.z, z.z); z.w = fmaf(s, v.w, z.w);
+    } else {
+      z.x += v.x; z.y += v.y; z.z += v.z; z.w += v.w;
+    }
+  }
+  if (b.extra) {
+    const float4 v = load4f((const AT*)b.extra + (size_t)t * H + 4 * gi);
+    z.x += v.x; z.y += v.y; z.z += v.z; z.w += v.w;
+  }
+  if (back != 0.f) {
+    const float4 v = load4f((const AT*)b.source + (size_t)t * H + 4 * gi);
+    z.x = fmaf(back, v.x, z.x); z.y = fmaf(back, v.y, z.y); z.z = fmaf(back, v.z, z.z); z.w = fmaf(back, v.w, z.w);
+  }
+  return z;
+}
+
+// out[t, :] = z of token t, for a consumer that wants one plain row
+template <typename AT>
+__global__ void __launch_bounds__(256) branch_sum_kernel(BranchArgs b, AT* __restrict__ out, long long n, int H) {
+  pdl_wait();
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n) return;
+  const int t = (int)(i / H);
+  out[i] = from_float<AT>(branch_at<AT>(b, t, H, (int)(i - (long long)t * H)));
+}
+
+// dst[t, :] = x[t, :] in the activation type; dst rows may lie further apart than their width.  With
+// a branch (b.rows), x[t, :] += z of token t first.
+template <typename AT>
+__global__ void __launch_bounds__(256)
+cast_rows_kernel(float* __restrict__ x, BranchArgs b, AT* __restrict__ dst, long long ld, long long n, int H) {
+  pdl_wait();
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n) return;
+  const int t = (int)(i / H), c = (int)(i - (long long)t * H);
+  float v = x[i];
+  if (b.rows) {
+    v += branch_at<AT>(b, t, H, c);
+    x[i] = v;
+  }
+  dst[t * ld + c] = from_float<AT>(v);
+}
+template <typename AT>
+__global__ void __launch_bounds__(256)
+cast_rows4_kernel(float* __restrict__ x, BranchArgs b, AT* __restrict__ dst, long long ld, long long n4, int groups) {
+  pdl_wait();
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n4) return;
+  const int t = (int)(i / groups), g = (int)(i - (long long)t * groups);
+  float4 v = load4f(x + 4 * i);
+  if (b.rows) {
+    const float4 z = branch_at4<AT>(b, t, 4 * groups, g);
+    v.x += z.x; v.y += z.y; v.z += z.z; v.w += z.w;
+    store4f(x + 4 * i, v);
+  }
+  store4f(dst + t * ld + 4 * g, v);
+}
+
+// ------------------------------------------------- a branch's own norm, then the residual
+// z as above; the residual takes mult * rms(z) * (w [+1]).  With a second weight the new residual
+// row is normed once more in the same pass and leaves as the next sublayer's input; with copy_out
+// it also leaves as it is, in the activation type.  A block owns a token; z, then the new residual
+// row, stay in shared memory (VEC: registers) between the passes.  `source` may be the buffer
+// that next_out writes: a block reads its token's row before its first sum, and writes it after.
 constexpr int NORM_ADD_KEEP = 8;   // groups of 4 elements a thread keeps between the passes
+
+struct NormAddArgs {
+  BranchArgs b;
+  const float* weight;
+  float* residual;
+  const float* next_weight;
+  void* next_out;
+  void* copy_out;
+  long long copy_ld;
+  int plus_one, next_plus_one, H;
+  float eps, next_eps, mult;
+};
 
 // VEC: rows of up to 4 * 256 * NORM_ADD_KEEP elements, a multiple of 4, every row 16-byte (bfloat16: 8-byte)
 // aligned: each row is read once, in 16-byte pieces, and stays in registers between the passes.
 template <typename AT, bool VEC>
-__global__ void __launch_bounds__(256)
-norm_add_kernel(const AT* __restrict__ branch, int k, const float* __restrict__ part_scale,
-                const float* __restrict__ weight, int plus_one, float eps, float mult,
-                float* __restrict__ residual, const float* __restrict__ next_weight, int next_plus_one,
-                float next_eps, AT* __restrict__ next_out, int H) {
+__global__ void __launch_bounds__(256) norm_add_kernel(NormAddArgs a) {
   extern __shared__ float row[];
   __shared__ float scratch[33];
   pdl_wait();
-  const int t = blockIdx.x;
-  const AT* b = branch + (size_t)t * k * H;
-  float* r = residual + (size_t)t * H;
-  const float one = plus_one ? 1.f : 0.f;
-  const float one2 = next_plus_one ? 1.f : 0.f;
+  const int t = blockIdx.x, H = a.H;
+  float* r = a.residual + (size_t)t * H;
+  const float one = a.plus_one ? 1.f : 0.f;
+  const float one2 = a.next_plus_one ? 1.f : 0.f;
+  const float mult = a.mult;
+  AT* copy = a.copy_out ? (AT*)a.copy_out + (size_t)t * a.copy_ld : nullptr;
+  AT* o = (AT*)a.next_out + (size_t)t * H;
   float ss = 0.f, ss2 = 0.f;
   if constexpr (VEC) {
     float4 keep[NORM_ADD_KEEP];
@@ -304,71 +422,58 @@ norm_add_kernel(const AT* __restrict__ branch, int k, const float* __restrict__ 
     for (int j = 0; j < NORM_ADD_KEEP; ++j) {
       const int gi = threadIdx.x + j * 256;
       if (gi < groups) {
-        float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
-        for (int q = 0; q < k; ++q) {
-          const float4 v = load4f(b + (size_t)q * H + 4 * gi);
-          if (part_scale) {
-            const float s = part_scale[q];
-            z.x = fmaf(s, v.x, z.x); z.y = fmaf(s, v.y, z.y); z.z = fmaf(s, v.z, z.z); z.w = fmaf(s, v.w, z.w);
-          } else {
-            z.x += v.x; z.y += v.y; z.z += v.z; z.w += v.w;
-          }
-        }
+        const float4 z = branch_at4<AT>(a.b, t, H, gi);
         keep[j] = z;
         ss = fmaf(z.x, z.x, ss); ss = fmaf(z.y, z.y, ss); ss = fmaf(z.z, z.z, ss); ss = fmaf(z.w, z.w, ss);
       }
     }
     ss = block_sum(ss, scratch);
-    const float inv = 1.0f / sqrtf(ss / (float)H + eps);
+    const float inv = 1.0f / sqrtf(ss / (float)H + a.eps);
 #pragma unroll
     for (int j = 0; j < NORM_ADD_KEEP; ++j) {
       const int gi = threadIdx.x + j * 256;
       if (gi < groups) {
-        const float4 w = load4f(weight + 4 * gi), x0 = load4f(r + 4 * gi), z = keep[j];
+        const float4 w = load4f(a.weight + 4 * gi), x0 = load4f(r + 4 * gi), z = keep[j];
         const float4 x = make_float4(x0.x + mult * (z.x * inv * (w.x + one)), x0.y + mult * (z.y * inv * (w.y + one)),
                                      x0.z + mult * (z.z * inv * (w.z + one)), x0.w + mult * (z.w * inv * (w.w + one)));
         store4f(r + 4 * gi, x);
+        if (copy) store4f(copy + 4 * gi, x);
         keep[j] = x;
         ss2 = fmaf(x.x, x.x, ss2); ss2 = fmaf(x.y, x.y, ss2); ss2 = fmaf(x.z, x.z, ss2); ss2 = fmaf(x.w, x.w, ss2);
       }
     }
-    if (!next_weight) return;
+    if (!a.next_weight) return;
     ss2 = block_sum(ss2, scratch);
-    const float inv2 = 1.0f / sqrtf(ss2 / (float)H + next_eps);
-    AT* o = next_out + (size_t)t * H;
+    const float inv2 = 1.0f / sqrtf(ss2 / (float)H + a.next_eps);
 #pragma unroll
     for (int j = 0; j < NORM_ADD_KEEP; ++j) {
       const int gi = threadIdx.x + j * 256;
       if (gi < groups) {
-        const float4 w = load4f(next_weight + 4 * gi), x = keep[j];
+        const float4 w = load4f(a.next_weight + 4 * gi), x = keep[j];
         store4f(o + 4 * gi, make_float4(x.x * inv2 * (w.x + one2), x.y * inv2 * (w.y + one2), x.z * inv2 * (w.z + one2),
                                         x.w * inv2 * (w.w + one2)));
       }
     }
-    return;
   } else {
-  for (int i = threadIdx.x; i < H; i += blockDim.x) {
-    float z = 0.f;
-    for (int j = 0; j < k; ++j) {
-      const float v = to_float(b[(size_t)j * H + i]);
-      z = part_scale ? fmaf(part_scale[j], v, z) : z + v;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+      const float z = branch_at<AT>(a.b, t, H, i);
+      row[i] = z;
+      ss = fmaf(z, z, ss);
     }
-    row[i] = z;
-    ss = fmaf(z, z, ss);
-  }
-  ss = block_sum(ss, scratch);
-  const float inv = 1.0f / sqrtf(ss / (float)H + eps);
-  for (int i = threadIdx.x; i < H; i += blockDim.x) {
-    const float x = r[i] + mult * (row[i] * inv * (weight[i] + one));
-    r[i] = x;
-    row[i] = x;
-    ss2 = fmaf(x, x, ss2);
-  }
-  if (!next_weight) return;
-  ss2 = block_sum(ss2, scratch);
-  const float inv2 = 1.0f / sqrtf(ss2 / (float)H + next_eps);
-  AT* o = next_out + (size_t)t * H;
-  for (int i = threadIdx.x; i < H; i += blockDim.x) o[i] = from_float<AT>(row[i] * inv2 * (next_weight[i] + one2));
+    ss = block_sum(ss, scratch);
+    const float inv = 1.0f / sqrtf(ss / (float)H + a.eps);
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+      const float x = r[i] + mult * (row[i] * inv * (a.weight[i] + one));
+      r[i] = x;
+      if (copy) copy[i] = from_float<AT>(x);
+      row[i] = x;
+      ss2 = fmaf(x, x, ss2);
+    }
+    if (!a.next_weight) return;
+    ss2 = block_sum(ss2, scratch);
+    const float inv2 = 1.0f / sqrtf(ss2 / (float)H + a.next_eps);
+    for (int i = threadIdx.x; i < H; i += blockDim.x)
+      o[i] = from_float<AT>(row[i] * inv2 * (a.next_weight[i] + one2));
   }
 }
 
@@ -892,23 +997,73 @@ int ft_softcap(float* x, long long n, float cap, cudaStream_t stream) {
   return FT_OK;
 }
 
-int ft_norm_add(const void* branch, int k, const float* part_scale, const float* weight, int plus_one, float eps,
+static int branch_args(BranchArgs& b, const void* rows, int k, const float* part_scale, const int* ids,
+                       const float* weights, int experts, const void* source, const void* extra) {
+  if (!rows || k <= 0 || (ids && (!weights || !source || part_scale || experts < 0))) return FT_ERR_SHAPE;
+  b = BranchArgs{rows, part_scale, ids, weights, source, extra, k, experts};
+  return FT_OK;
+}
+
+int ft_norm_add(const void* branch, int k, const float* part_scale, const int* ids, const float* route_weights,
+                int experts, const void* source, const void* extra, const float* weight, int plus_one, float eps,
                 float mult, float* residual, const float* next_weight, int next_plus_one, float next_eps,
-                void* next_out, int T, int H, int dtype, cudaStream_t stream) {
+                void* next_out, void* copy_out, long long copy_ld, int T, int H, int dtype, cudaStream_t stream) {
   if (T <= 0) return FT_OK;
-  if (k <= 0 || H <= 0 || H > 12288) return FT_ERR_SHAPE;
+  NormAddArgs a{};
+  const int rc = branch_args(a.b, branch, k, part_scale, ids, route_weights, experts, source, extra);
+  if (rc != FT_OK) return rc;
+  if (H <= 0 || H > 12288) return FT_ERR_SHAPE;
+  a.weight = weight; a.residual = residual; a.next_weight = next_weight; a.next_out = next_out;
+  a.copy_out = copy_out; a.copy_ld = copy_ld; a.plus_one = plus_one; a.next_plus_one = next_plus_one; a.H = H;
+  a.eps = eps; a.next_eps = next_eps; a.mult = mult;
   const bool vec = !(H & 3) && H <= 4 * 256 * NORM_ADD_KEEP && !((uintptr_t)branch & 15) && !((uintptr_t)weight & 15) &&
-                   !((uintptr_t)residual & 15) && !((uintptr_t)next_weight & 15) && !((uintptr_t)next_out & 15);
+                   !((uintptr_t)residual & 15) && !((uintptr_t)next_weight & 15) && !((uintptr_t)next_out & 15) &&
+                   !((uintptr_t)source & 15) && !((uintptr_t)extra & 15) && !((uintptr_t)copy_out & 15) &&
+                   !(copy_ld & 3);
   if (vec) {
-    FT_DISPATCH(dtype, AT,
-                (launch_pdl(norm_add_kernel<AT, true>, dim3(T), dim3(256), 0, stream, (const AT*)branch, k, part_scale,
-                            weight, plus_one, eps, mult, residual, next_weight, next_plus_one, next_eps,
-                            (AT*)next_out, H)));
+    FT_DISPATCH(dtype, AT, (launch_pdl(norm_add_kernel<AT, true>, dim3(T), dim3(256), 0, stream, a)));
   } else {
     FT_DISPATCH(dtype, AT,
-                (launch_pdl(norm_add_kernel<AT, false>, dim3(T), dim3(256), (size_t)H * sizeof(float), stream,
-                            (const AT*)branch, k, part_scale, weight, plus_one, eps, mult, residual, next_weight,
-                            next_plus_one, next_eps, (AT*)next_out, H)));
+                (launch_pdl(norm_add_kernel<AT, false>, dim3(T), dim3(256), (size_t)H * sizeof(float), stream, a)));
+  }
+  FT_LAUNCH_CHECK();
+  return FT_OK;
+}
+
+int ft_branch_sum(const void* branch, int k, const int* ids, const float* route_weights, int experts,
+                  const void* source, const void* extra, void* out, int T, int H, int dtype, cudaStream_t stream) {
+  if (T <= 0) return FT_OK;
+  BranchArgs b;
+  const int rc = branch_args(b, branch, k, nullptr, ids, route_weights, experts, source, extra);
+  if (rc != FT_OK) return rc;
+  const long long n = (long long)T * H;
+  FT_DISPATCH(dtype, AT,
+              (launch_pdl(branch_sum_kernel<AT>, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, b,
+                          (AT*)out, n, H)));
+  FT_LAUNCH_CHECK();
+  return FT_OK;
+}
+
+int ft_cast_rows(float* x, const void* branch, int k, const int* ids, const float* route_weights, int experts,
+                 const void* source, const void* extra, void* dst, long long ld, int T, int H, int dtype,
+                 cudaStream_t stream) {
+  if (T <= 0 || H <= 0) return FT_OK;
+  BranchArgs b{};
+  if (branch) {
+    const int rc = branch_args(b, branch, k, nullptr, ids, route_weights, experts, source, extra);
+    if (rc != FT_OK) return rc;
+  }
+  const long long n = (long long)T * H;
+  const int groups = H / 4;
+  if (!(H & 3) && !(ld & 3) && !((uintptr_t)x & 15) && !((uintptr_t)dst & 15) && !((uintptr_t)branch & 15) &&
+      !((uintptr_t)source & 15) && !((uintptr_t)extra & 15)) {
+    FT_DISPATCH(dtype, AT,
+                (launch_pdl(cast_rows4_kernel<AT>, dim3((unsigned)((n / 4 + 255) / 256)), dim3(256), 0, stream, x, b,
+                            (AT*)dst, ld, n / 4, groups)));
+  } else {
+    FT_DISPATCH(dtype, AT,
+                (launch_pdl(cast_rows_kernel<AT>, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, x, b,
+                            (AT*)dst, ld, n, H)));
   }
   FT_LAUNCH_CHECK();
   return FT_OK;

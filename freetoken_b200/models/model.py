@@ -1,6 +1,6 @@
 """The generic decoder: parts built from a plan, run in the plan's order.
 
-``embed -> for stop in schedule: block(stop.layer) -> final norm -> head`` with
+``embed -> for stop in schedule: [stream map,] block(stop.layer) -> final norm -> head`` with
 the ``(delta, residual)`` pair carried between blocks
 (python/freetoken/models/minimax_m2/model.py:48-52,66-68).  The model owns no
 sizes and no cache: parts carry their parameters, the engine hands each stop
@@ -16,8 +16,8 @@ import torch
 from ..cache.manager import CacheNeed
 from ..config.model_plan import ModelPlan, PartSpec
 from ..csrc import ops
-from ..parts.base import (BLOCKS, EMBEDDINGS, FEED_FORWARDS, HEADS, MIXERS, NORMS, Block, CacheView, Part,
-                          StepContext)
+from ..parts.base import (BLOCKS, EMBEDDINGS, FEED_FORWARDS, HEADS, MIXERS, NORMS, STREAM_MAPS, Block,
+                          CacheView, Part, StepContext, StreamMap)
 from ..weights.spec import TensorSpec
 
 
@@ -56,6 +56,8 @@ class Model:
                 ffn = FEED_FORWARDS.get(layer.feed_forward.kind)(layer.feed_forward, layer.prefix)
             norms = {name: NORMS.get(spec.kind)(spec, layer.prefix) for name, spec in norm_specs.items()}
             self.blocks.append(block_cls(layer.block, layer.prefix, mixer, ffn, norms))
+        self.stream_maps: List[StreamMap] = [STREAM_MAPS.get(spec.kind)(spec, _prefix(spec, ""))
+                                             for spec in plan.stream_maps]
         self.final_norm = NORMS.get(plan.final_norm.kind)(plan.final_norm, _prefix(plan.final_norm, ""))
         self.head = HEADS.get(plan.head.kind)(plan.head, _prefix(plan.head, ""))
         if nvtx:
@@ -63,12 +65,14 @@ class Model:
                 _with_nvtx_range(block, f"layer_{i}")
                 for child in block.children():
                     _with_nvtx_range(child, f"layer_{i}.{type(child).__name__}")
+            for i, part in enumerate(self.stream_maps):
+                _with_nvtx_range(part, f"stream_map_{i}")
             for part, name in ((self.embedding, "embedding"), (self.final_norm, "final_norm"), (self.head, "head")):
                 _with_nvtx_range(part, name)
 
     # ---- weights ---------------------------------------------------------
     def parts(self):
-        return [self.embedding, *self.blocks, self.final_norm, self.head]
+        return [self.embedding, *self.blocks, *self.stream_maps, self.final_norm, self.head]
 
     def tensor_specs(self) -> List[TensorSpec]:
         specs: List[TensorSpec] = []
@@ -150,8 +154,13 @@ class Model:
             self.embedding.forward(ctx, residual, caches[len(self.plan.schedule)])
         else:
             self.embedding.forward(ctx, residual)
+        for part in self.stream_maps:
+            part.begin(ctx, residual)
         delta = None
         for stop, cache in zip(self.plan.schedule, caches):
+            if stop.stream_map is not None:
+                self.stream_maps[stop.stream_map].forward(ctx, delta, residual)
+                delta = None
             delta = self.blocks[stop.layer].forward(ctx, delta, residual, cache)
         n = logit_rows.numel()
         if n == 0:

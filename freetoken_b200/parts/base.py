@@ -20,6 +20,8 @@ Kinds of parts and what each must offer:
 * **Block**         arranges a mixer, a feed-forward (if it has one) and the
   norms it names around the residual stream:
   ``forward(ctx, delta, residual, cache) -> delta``.
+* **StreamMap**     ``forward(ctx, delta, residual)`` in front of a stop of the schedule
+  that asks for it: joins the pending branch and replaces the residual rows.
 
 Any part whose kernels want step metadata of their own (row lists, tile lists)
 states a ``step_plan_key()`` and builds the lists in ``plan_step(shape)``; the
@@ -325,6 +327,18 @@ class Block(Part):
         raise NotImplementedError
 
 
+class StreamMap(Part):
+    """Something that happens to the residual stream between two layers: ``forward`` joins what the
+    layer before left pending and replaces the stream's rows.  ``begin`` is called once a step, with
+    the stream as the embedding left it."""
+
+    def begin(self, ctx: StepContext, residual: torch.Tensor) -> None:
+        pass
+
+    def forward(self, ctx: StepContext, delta, residual: torch.Tensor) -> None:
+        raise NotImplementedError
+
+
 class Embedding(Part):
     def cache_need(self) -> Optional[CacheNeed]:
         """What the cache manager keeps per request for the embedding (a ``PerRequestNeed``), or
@@ -372,6 +386,7 @@ FEED_FORWARDS = Registry("feed-forward")
 BLOCKS = Registry("block")
 EMBEDDINGS = Registry("embedding")
 HEADS = Registry("head")
+STREAM_MAPS = Registry("stream map")
 
 register_norm = NORMS.register
 register_position = POSITIONS.register
@@ -380,3 +395,4 @@ register_feed_forward = FEED_FORWARDS.register
 register_block = BLOCKS.register
 register_embedding = EMBEDDINGS.register
 register_head = HEADS.register
+register_stream_map = STREAM_MAPS.register

@@ -28,8 +28,9 @@ joins the residual stream::
     residual += mult * norm_out'(feed_forward(norm_in'(residual)))
 
 Both sums happen in float32 inside the norm kernel that computes the output norm; the
-output norm of the mixer and the input norm of the feed-forward are one launch.  The
-block leaves nothing pending (it returns ``None``).
+output norm of the mixer and the input norm of the feed-forward are one launch.  The last
+sublayer's output leaves the block pending, with its norm (:class:`~.norm.NormedBranch`): the
+next layer's first norm (or the last norm) joins it and norms the sum in one launch.
 
 ``hyper`` is a pre-norm block over several residual streams (hyper-connections): each of its
 norms (:class:`~.norm.HyperNorm`) forms its sublayer's input from all streams and owns the weights
@@ -45,6 +46,7 @@ next such norm folds in::
 from __future__ import annotations
 
 from .base import Block, register_block
+from .norm import NormedBranch, plain_branch
 
 
 @register_block("prenorm")
@@ -83,7 +85,7 @@ class ParallelBlock(Block):
         if self.feed_forward.writes_into_out:
             self.feed_forward.forward(ctx, h, out=pair[:, 1])
         else:
-            pair[:, 1].copy_(self.feed_forward.forward(ctx, h))
+            pair[:, 1].copy_(plain_branch(ctx, self.feed_forward.forward(ctx, h)))
         return pair
 
 
@@ -109,12 +111,9 @@ class SandwichBlock(Block):
         h = self.norms["mixer"].forward(ctx, delta, residual)
         a = self.mixer.forward(ctx, h, cache)
         if self.feed_forward is None:
-            self.norms["mixer_out"].add_normed(ctx, a, residual, self.mult)
-            return None
+            return NormedBranch(a, self.norms["mixer_out"], self.mult)
         h = self.norms["mixer_out"].add_normed(ctx, a, residual, self.mult, then=self.norms["feed_forward"])
-        f = self.feed_forward.forward(ctx, h)
-        self.norms["feed_forward_out"].add_normed(ctx, f, residual, self.mult)
-        return None
+        return NormedBranch(self.feed_forward.forward(ctx, h), self.norms["feed_forward_out"], self.mult)
 
 
 @register_block("hyper")

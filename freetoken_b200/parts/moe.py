@@ -11,6 +11,11 @@ python/freetoken/layers/moe.py:83-92): routes are sorted by expert;
 ``m = act(Wgate_e x) * (Wup_e x)`` from one product against ``[gate; up]``;
 ``y_route = w_route * (Wdown_e m)`` with the weight applied to the float32
 accumulator; ``y = sum over the k routes`` in float32, slot order.
+Two options no model of the reference has: ``identity`` - the last outputs of the router stand for
+experts without weights that hand the input back, times the route's weight (their routes are sorted
+behind all others and no product touches them) - and ``shared``, a gated feed-forward every token
+passes, added.  With either the result is :class:`ops.RoutedRows`: the consumer's kernel adds the
+routed rows, the handed-back input and the shared row in float32, in one pass.
 Activation ``silu`` or ``swigluoai``
 (python/freetoken/kernel/triton/activation.py:96-107).
 """
@@ -24,7 +29,7 @@ import torch
 from ..csrc import ops
 from ..weights.spec import Cat, Init, Name, Stack, TensorSpec
 from . import linear
-from .base import FeedForward, StepContext, register_feed_forward
+from .base import FEED_FORWARDS, FeedForward, StepContext, register_feed_forward
 
 
 # Above this many rows per expert (on average) the experts run on the tcgen05
@@ -65,7 +70,9 @@ class RoutedExperts(FeedForward):
     down_each: per-expert checkpoint names with ``{e}``).  ``groups`` and ``keep_groups``
     (default 1, 1: no groups): the experts form ``groups`` equal groups of neighbours, a group's
     value is the sum of its two largest choice scores (score plus bias), and only experts of the
-    ``keep_groups`` best groups can be chosen."""
+    ``keep_groups`` best groups can be chosen.  ``identity`` (default 0): so many router outputs behind
+    the ``num_experts`` experts' hand the input back.  ``shared`` (a PartSpec of a feed-forward, or
+    None): one that runs for every token beside the routed experts."""
 
     graph_capturable = True
 
@@ -83,14 +90,21 @@ class RoutedExperts(FeedForward):
         self.act = p.get("activation", "silu")
         self.act_alpha = float(p.get("act_alpha", 1.702))
         self.act_limit = float(p.get("act_limit", 7.0))
-        if self.k > self.E:
-            raise ValueError(f"top_k {self.k} exceeds num_experts {self.E}")
+        self.identity = int(p.get("identity") or 0)
+        self.outputs = self.E + self.identity          # of the router
+        if self.k > self.outputs:
+            raise ValueError(f"top_k {self.k} exceeds the router's {self.outputs} outputs")
         self.groups = int(p.get("groups", 1))
         self.keep_groups = int(p.get("keep_groups", self.groups))
-        if (self.groups < 1 or self.E % self.groups or not 1 <= self.keep_groups <= self.groups
-                or self.keep_groups * (self.E // self.groups) < self.k or self.groups > 256):
+        if (self.groups < 1 or self.outputs % self.groups or not 1 <= self.keep_groups <= self.groups
+                or self.keep_groups * (self.outputs // self.groups) < self.k or self.groups > 256):
             raise ValueError(f"{self.groups} groups of which {self.keep_groups} are kept do not fit "
-                             f"{self.E} experts, top-{self.k}")
+                             f"{self.outputs} experts, top-{self.k}")
+        self.shared = None
+        if p.get("shared") is not None:
+            self.shared = FEED_FORWARDS.get(p["shared"].kind)(p["shared"], prefix)
+            if not self.shared.writes_into_out:
+                raise ValueError("the shared feed-forward must be able to leave its result in a given place")
         names = p["checkpoint_names"]
         self.scope = self.name(p["scope"])
         self.n_router = f"{self.scope}.{names['router']}"
@@ -100,6 +114,9 @@ class RoutedExperts(FeedForward):
         self._each = {key: f"{self.scope}.{names[key]}" for key in ("gate", "up", "down_each")}
         self.w_router = self.w_router_terms = self.w_bias = self.w_gate_up = self.w_down = None
 
+    def children(self):
+        return [self.shared] if self.shared is not None else []
+
     def tensor_specs(self) -> List[TensorSpec]:
         E, I, H = self.E, self.inter, self.hidden
         gate_up = Stack(tuple(
@@ -107,13 +124,13 @@ class RoutedExperts(FeedForward):
                  Name(self._each["up"].format(e=e), (I, H))), 0) for e in range(E)))
         down = Stack(tuple(Name(self._each["down_each"].format(e=e), (H, I)) for e in range(E)))
         return [
-            TensorSpec(self.n_router, (E, H), role="small32", keep_float32_in_file=True),
-            TensorSpec(self.n_bias, (E,), role="small32", keep_float32_in_file=True,
+            TensorSpec(self.n_router, (self.outputs, H), role="small32", keep_float32_in_file=True),
+            TensorSpec(self.n_bias, (self.outputs,), role="small32", keep_float32_in_file=True,
                        init=Init(0.0, 0.01 if self.use_bias else 0.0), tag="router_bias",
                        optional=not self.use_bias),
             TensorSpec(self.n_gate_up, (E, 2 * I, H), sources=(gate_up,)),
             TensorSpec(self.n_down, (E, H, I), sources=(down,), tag="residual_out"),
-        ]
+        ] + (self.shared.tensor_specs() if self.shared is not None else [])
 
     def bind(self, tensors: Dict[str, torch.Tensor], dtype) -> None:
         self.w_router = tensors[self.n_router]
@@ -124,9 +141,12 @@ class RoutedExperts(FeedForward):
         self.w_bias = tensors.get(self.n_bias)
         self.w_gate_up = tensors[self.n_gate_up]
         self.w_down = tensors[self.n_down]
+        if self.shared is not None:
+            self.shared.bind(tensors, dtype)
 
     def libraries(self, dtype) -> List[str]:
-        libs = ["gemm_simt", "moe_route", "elementwise"]
+        libs = ["gemm_simt", "moe_route", "elementwise"] + (["rowwise"] if self.identity or self.shared else [])
+        libs += [lib for lib in (self.shared.libraries(dtype) if self.shared else []) if lib not in libs]
         return libs + (["skinny_gemm", "moe_gemm_tc"] if dtype == torch.bfloat16 else [])
 
     # ---- forward ----------------------------------------------------------------
@@ -137,7 +157,7 @@ class RoutedExperts(FeedForward):
         whether that was done here (a handful of tokens: one launch for both)."""
         T = x.shape[0]
         ws = ctx.workspace
-        logits = ws.get("moe.logits", (T, self.E), torch.float32)
+        logits = ws.get("moe.logits", (T, self.outputs), torch.float32)
         terms = 1
         if ctx.dtype == torch.bfloat16 and T <= ROUTER_SMALL_T and ops.router_logits_takes(x, self.w_router):
             ops.router_logits(x, self.w_router, logits)
@@ -146,26 +166,26 @@ class RoutedExperts(FeedForward):
                                                torch.float32)):
             # many rows: tensor-core products of the bfloat16 activations with the exact
             # bfloat16 terms of the float32 router weight; the terms are summed by the selection
-            terms = self.w_router_terms.shape[0] // self.E
+            terms = self.w_router_terms.shape[0] // self.outputs
             logits = ws.get("moe.logit_terms", (T, self.w_router_terms.shape[0]), torch.float32)
         else:
             ops.gemm_rows(x, self.w_router, logits)
         ids = ws.get("moe.ids", (T, self.k), torch.int32)
         weights = ws.get("moe.weights", (T, self.k), torch.float32)
-        if sort_into is not None and ops.route_small_takes(T, self.E, self.k):
+        if sort_into is not None and ops.route_small_takes(T, self.outputs, self.k):
             ops.route_small(logits, self.w_bias, ids, weights, *sort_into, self.k, self.softmax,
-                            self.renorm, self.scale, terms, self.groups, self.keep_groups)
+                            self.renorm, self.scale, terms, self.groups, self.keep_groups, busy_of=self.E)
             return ids, weights, True
         ops.router_select(logits, self.w_bias, ids, weights, self.k, self.softmax, self.renorm,
                           self.scale, terms, self.groups, self.keep_groups)
         return (ids, weights) if sort_into is None else (ids, weights, False)
 
-    def forward(self, ctx: StepContext, x: torch.Tensor) -> torch.Tensor:
+    def forward(self, ctx: StepContext, x: torch.Tensor):
         T = x.shape[0]
         R = T * self.k
         ws = ctx.workspace
-        counts = ws.get("moe.counts", (self.E,), torch.int32)
-        offsets = ws.get("moe.offsets", (self.E + 1,), torch.int32)
+        counts = ws.get("moe.counts", (self.outputs,), torch.int32)
+        offsets = ws.get("moe.offsets", (self.outputs + 1,), torch.int32)
         sorted_route = ws.get("moe.sorted_route", (R,), torch.int32)
         sorted_token = ws.get("moe.sorted_token", (R,), torch.int32)
         active = ws.get("moe.active", (self.E + 1,), torch.int32)
@@ -173,21 +193,29 @@ class RoutedExperts(FeedForward):
         if not is_sorted:
             scratch = None
             if R >= ops.MOE_SORT_CHUNKED_FROM:
-                scratch = ws.get("moe.sort_scratch", (ops.moe_sort_scratch(R, self.E),), torch.int32)
-            ops.moe_sort(ids.view(-1), counts, offsets, sorted_route, sorted_token, active, self.E,
-                         self.k, scratch)
+                scratch = ws.get("moe.sort_scratch", (ops.moe_sort_scratch(R, self.outputs),), torch.int32)
+            ops.moe_sort(ids.view(-1), counts, offsets, sorted_route, sorted_token, active, self.outputs,
+                         self.k, scratch, busy_of=self.E)
         if ctx.probe is not None:
             if "router_ids" in ctx.probe:
                 ctx.probe["router_ids"].append(ids.clone())
             else:
-                ctx.probe.setdefault("experts_touched", []).append(int((counts > 0).sum()))
+                ctx.probe.setdefault("experts_touched", []).append(int((counts[:self.E] > 0).sum()))
         mid = ws.get("moe.mid", (R, self.inter), ctx.dtype)
         parts = ws.get("moe.parts", (R, self.hidden), ctx.dtype)
         self.experts(ctx, x, mid, parts, offsets, active, sorted_route, sorted_token,
                      weights.view(-1), R)
         # the k partial rows of a token are summed by whoever consumes them
         # (the next norm adds them into the residual in slot order)
-        return parts.view(T, self.k, self.hidden)
+        parts = parts.view(T, self.k, self.hidden)
+        if self.shared is None and not self.identity:
+            return parts
+        extra = None
+        if self.shared is not None:
+            extra = self.shared.forward(ctx, x, out=ws.get("moe.shared", (T, self.hidden), ctx.dtype))
+        if not self.identity:
+            return ops.RoutedRows(parts, extra=extra)
+        return ops.RoutedRows(parts, ids, weights, self.E, x, extra)
 
     def experts(self, ctx, x, mid, parts, offsets, active, sorted_route, sorted_token, route_weight, R):
         if ctx.dtype == torch.bfloat16 and R > TC_MIN_ROWS_PER_EXPERT * self.E \

@@ -21,7 +21,9 @@ from .base import Norm, StepContext, register_norm
 @register_norm("rmsnorm")
 class RMSNorm(Norm):
     """params: ``size``, ``eps``, ``plus_one``, and ``scope`` (the tensor is ``<scope>.weight``
-    below the prefix) or ``tensor`` (its whole name below the prefix)."""
+    below the prefix) or ``tensor`` (its whole name below the prefix).  ``scale_tensor`` (None: none):
+    a second vector the normed values are multiplied by element by element (a layer scale behind a
+    sublayer's output norm); the product of both vectors is formed once, in float32, at binding."""
 
     graph_capturable = True
 
@@ -31,36 +33,79 @@ class RMSNorm(Norm):
         self.eps = float(spec.params["eps"])
         self.plus_one = bool(spec.get("plus_one", False))
         self.weight_name = self.name(spec.get("tensor") or f"{spec.params['scope']}.weight")
+        self.scale_name = self.name(spec.get("scale_tensor")) if spec.get("scale_tensor") else None
+        if self.scale_name and self.plus_one:
+            raise ValueError("a scale beside a one-plus norm weight is not offered")
         self.weight: Optional[torch.Tensor] = None
 
     def tensor_specs(self) -> List[TensorSpec]:
         mean = 0.0 if self.plus_one else 1.0
-        return [TensorSpec(self.weight_name, (self.size,), role="small32",
-                           init=Init(mean=mean, std=0.0), tag="norm")]
+        return [TensorSpec(name, (self.size,), role="small32", init=Init(mean=mean, std=0.0), tag="norm")
+                for name in (self.weight_name, self.scale_name) if name]
 
     def bind(self, tensors: Dict[str, torch.Tensor], dtype) -> None:
         self.weight = tensors[self.weight_name]
+        if self.scale_name:
+            self.weight = self.weight * tensors[self.scale_name]
 
     def libraries(self, dtype) -> List[str]:
         return ["elementwise", "rowwise"]
 
     def forward(self, ctx: StepContext, delta, residual: torch.Tensor) -> torch.Tensor:
+        if isinstance(delta, NormedBranch):
+            # the branch's own norm, the sum and this norm in one launch
+            return delta.norm.add_normed(ctx, delta.y, residual, delta.mult, then=self)
         out = ctx.workspace.get("norm.out", residual.shape, ctx.dtype)
-        ops.rmsnorm(delta, residual, self.weight, out, self.eps, self.plus_one)
+        ops.rmsnorm(plain_branch(ctx, delta), residual, self.weight, out, self.eps, self.plus_one)
         return out
 
-    def add_normed(self, ctx: StepContext, branch: torch.Tensor, residual: torch.Tensor, mult: float,
-                   then: Optional["RMSNorm"] = None) -> Optional[torch.Tensor]:
+    def add_normed(self, ctx: StepContext, branch, residual: torch.Tensor, mult: float,
+                   then: Optional["RMSNorm"] = None, copy_out: Optional[torch.Tensor] = None
+                   ) -> Optional[torch.Tensor]:
         """``residual += mult * norm(branch)`` in float32, this norm being the branch's own
-        (``branch`` is ``[T, H]`` or ``[T, k, H]`` partial rows, summed first).  With ``then`` the
-        new residual rows are normed by that norm in the same launch and returned."""
+        (``branch`` is ``[T, H]`` or ``[T, k, H]`` partial rows or :class:`ops.RoutedRows`, summed first).
+        With ``then`` the new residual rows are normed by that norm in the same launch and returned;
+        with ``copy_out`` they also leave as they are, in the activation type."""
         if then is None:
-            ops.norm_add(branch, residual, self.weight, self.eps, self.plus_one, mult)
+            ops.norm_add(branch, residual, self.weight, self.eps, self.plus_one, mult, copy_out=copy_out)
             return None
         out = ctx.workspace.get("norm.out", residual.shape, ctx.dtype)
         ops.norm_add(branch, residual, self.weight, self.eps, self.plus_one, mult, next_weight=then.weight,
-                     next_eps=then.eps, next_plus_one=then.plus_one, next_out=out)
+                     next_eps=then.eps, next_plus_one=then.plus_one, next_out=out, copy_out=copy_out)
         return out
+
+
+class NormedBranch:
+    """A sublayer's output that has not joined the residual stream yet and passes a norm of its own
+    first: ``x <- x + mult * norm(y)``.  A sandwich block hands it on where other blocks hand on a plain
+    branch output; the next :class:`RMSNorm` (the next layer's or the model's last) folds it in with
+    its own norm in one launch, :func:`add_pending` does it where no norm follows."""
+
+    __slots__ = ("y", "norm", "mult")
+
+    def __init__(self, y, norm: "RMSNorm", mult: float):
+        self.y, self.norm, self.mult = y, norm, mult
+
+
+def plain_branch(ctx: StepContext, delta):
+    """``delta`` as a tensor of (partial) rows: a routed feed-forward's unsummed result is summed."""
+    if isinstance(delta, ops.RoutedRows):
+        rows = delta.rows
+        out = ctx.workspace.get("norm.branch", (rows.shape[0], rows.shape[-1]), ctx.dtype)
+        ops.branch_sum(delta, out)
+        return out
+    return delta
+
+
+def add_pending(ctx: StepContext, delta, residual: torch.Tensor, copy_out: torch.Tensor) -> None:
+    """Whatever a block left pending joins the plain residual stream; the new rows also leave, in the
+    activation type, through ``copy_out`` (``[T, H]``, rows may lie further apart)."""
+    if isinstance(delta, NormedBranch):
+        delta.norm.add_normed(ctx, delta.y, residual, delta.mult, copy_out=copy_out)
+        return
+    if isinstance(delta, PendingBranch):
+        raise ValueError("a branch with connection weights joins several streams, not the plain residual")
+    ops.cast_rows(residual, copy_out, delta)
 
 
 class PendingBranch:
@@ -148,6 +193,6 @@ class HyperNorm(Norm):
                              "(PendingBranch), not as a plain tensor")
         T, _, H = residual.shape
         out = ctx.workspace.get("norm.out", (T, H), ctx.dtype)
-        y, mix, w_out = (delta.y, delta.mix, delta.out) if delta is not None else (None, None, None)
+        y, mix, w_out = (plain_branch(ctx, delta.y), delta.mix, delta.out) if delta is not None else (None, None, None)
         ops.hyper_norm(residual, y, mix, w_out, self.w_in, self.weight, self.bias, self.eps, self.center, out)
         return out

@@ -141,3 +141,12 @@ def _load_builtin() -> None:
             config_to_dict=lambda cfg: cfg.to_dict(),
         ),
     )
+    from .config import dizatar
+    register_architecture(
+        Architecture(
+            name=dizatar.ARCHITECTURE,
+            read_config=dizatar.DizatarConfig.from_dict,
+            build_plan=dizatar.build_plan,
+            config_to_dict=lambda cfg: cfg.to_dict(),
+        ),
+    )
