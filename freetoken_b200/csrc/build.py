@@ -46,6 +46,8 @@ LIBRARIES: Dict[str, str] = {
     "attention_decode_tma": "attention_decode_tma.cu",
     "attention_prefill": "attention_prefill.cu",
     "attention_prefill_tc": "attention_prefill_tc.cu",
+    "attention_latent": "attention_latent.cu",
+    "attention_prefill_mha": "attention_prefill_mha.cu",
     "moe_gemm_tc": "moe_gemm_tc.cu",
     "recurrent": "recurrent.cu",
 }

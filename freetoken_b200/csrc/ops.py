@@ -536,25 +536,27 @@ def rms_rows(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, eps: floa
              _stream()), "rms_rows")
 
 
-def latent_store(down: torch.Tensor, q: torch.Tensor, q_abs: torch.Tensor, pages: Optional[torch.Tensor],
+def latent_store(down: torch.Tensor, q: torch.Tensor, q_abs: Optional[torch.Tensor], pages: Optional[torch.Tensor],
                  weight: torch.Tensor, cos_sin: Optional[torch.Tensor], token_pos: torch.Tensor,
                  token_seg: torch.Tensor, block_table: torch.Tensor, *, heads: int, q_dim: int, rank: int,
-                 rot: int, interleaved: bool, eps: float) -> None:
+                 rot: int, interleaved: bool, eps: float, turn_q: bool = False) -> None:
     """Latent attention with a rotated key part, between projections and attention.  ``down`` rows are
     ``[latent (rank) | key part (rot)]``: the latent is RMS-normed times ``weight``, the key part turned
     by the token's position, both stored as one row ``[rank + rot]`` of ``pages`` (``[pages, 1, page,
     rank + rot]``; None: nothing is stored).  ``q`` rows hold ``heads`` times ``[q_dim | rot]``: every
     head's last ``rot`` values are turned and written behind the first ``rank`` values of its row of
-    ``q_abs`` (``[T, heads, rank + rot]``)."""
+    ``q_abs`` (``[T, heads, rank + rot]``; None: nowhere); with ``turn_q`` the turned values also take
+    their own place in ``q``."""
     _need(down, "down", contiguous=False)
     _need(q, "q", down.dtype, contiguous=False)
-    _need(q_abs, "q_abs", down.dtype)
+    if q_abs is not None:
+        _need(q_abs, "q_abs", down.dtype)
     _need(weight, "weight", torch.float32)
     for name, t in (("token_pos", token_pos), ("token_seg", token_seg), ("block_table", block_table)):
         _need(t, name, torch.int32)
     T = down.shape[0]
     if down.shape[1] != rank + rot or q.shape != (T, heads * (q_dim + rot)) or down.stride(1) != 1 \
-            or q.stride(1) != 1 or q_abs.shape != (T, heads, rank + rot) or weight.numel() != rank:
+            or q.stride(1) != 1 or (q_abs is not None and q_abs.shape != (T, heads, rank + rot)) or weight.numel() != rank:
         raise KernelError("latent_store: shapes do not match")
     if rot:
         _need(cos_sin, "cos_sin", torch.float32)
@@ -566,10 +568,10 @@ def latent_store(down: torch.Tensor, q: torch.Tensor, q_abs: torch.Tensor, pages
         if pages.dim() != 4 or pages.shape[1] != 1 or pages.shape[3] != rank + rot:
             raise KernelError("latent_store: pages must be [pages, 1, page, rank + rot]")
         P, page_stride = pages.shape[2], pages.stride(0)
-    f = _fn("rowwise", "ft_latent_store", "p q p q p p q p p p p p i i i i i i i f i i")
+    f = _fn("rowwise", "ft_latent_store", "p q p q p p q p p p p p i i i i i i i i f i i")
     _check(f(_ptr(down), down.stride(0), _ptr(q), q.stride(0), _ptr(q_abs), _ptr(pages), page_stride, _ptr(weight),
              _ptr(cos_sin), _ptr(token_pos), _ptr(token_seg), _ptr(block_table), heads, q_dim, rank, rot, P,
-             block_table.shape[1], int(interleaved), float(eps), code(down.dtype), T, _stream()), "latent_store")
+             block_table.shape[1], int(interleaved), int(turn_q), float(eps), code(down.dtype), T, _stream()), "latent_store")
 
 
 # ------------------------------------------------------- mixers with a carried state
@@ -1275,6 +1277,148 @@ def attn_prefill_tc(q: torch.Tensor, out: torch.Tensor, kv_pages: torch.Tensor,
              _ptr(status), num_heads, num_kv_heads, head_dim, kv_pages.shape[3], block_table.shape[1],
              tile_seg.numel(), float(scale), 1 if kv_pages.stride(0) else 0, int(window or 0),
              *(options or NO_SCORE_OPTIONS).args(num_heads), _stream()), "attn_prefill_tc")
+
+
+# ------------------------------------------- attention over latent rows, absorbed and expanded
+LATENT_KEYS = 64       # keys per tile of the absorbed kernel
+LATENT_MERGE_COST = 3  # what the merge of its splits costs, in tiles
+
+
+def attn_latent_takes(dtype: torch.dtype, d: int, rank: int) -> bool:
+    """Rows of any multiple of 8 up to 1,024 values, of which a multiple of 8 are the value (bfloat16)."""
+    return dtype == torch.bfloat16 and d % 8 == 0 and rank % 8 == 0 and 0 < rank <= d <= 1024
+
+
+def latent_row_tile(num_heads: int) -> int:
+    """Flat query rows (token-major, then head) per CTA: 16, or 32 where a token has more heads."""
+    return 16 if num_heads <= 16 else 32
+
+
+def latent_splits(tiles: int, max_kv_len: int, slots: int) -> tuple:
+    """``(splits, keys per split)`` with the least rounds of CTAs x (tiles per split + a CTA's fixed cost)."""
+    key_tiles = max(1, -(-max_kv_len // LATENT_KEYS))
+    best, best_cost = 1, None
+    for want in range(1, min(key_tiles, 64) + 1):
+        per = -(-key_tiles // want)
+        if -(-key_tiles // per) != want:
+            continue
+        cost = -(-tiles * want // slots) * (per + 3) + (LATENT_MERGE_COST if want > 1 else 0)
+        if best_cost is None or cost < best_cost:
+            best, best_cost = want, cost
+    per = -(-key_tiles // best)
+    return -(-key_tiles // per), per * LATENT_KEYS
+
+
+def attn_latent(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, tile_seg: torch.Tensor,
+                tile_row: torch.Tensor, seg_q_start: torch.Tensor, seg_pos0: torch.Tensor,
+                block_table: torch.Tensor, num_heads: int, rank: int, scale: float, window: Optional[int],
+                max_kv_len: int, workspace) -> None:
+    """Attention of absorbed queries ``q`` ``[T, heads, d]`` over cached rows ``pages`` ``[pages, 1, page, d]``
+    whose first ``rank`` values are also the value; ``out`` ``[T, heads, rank]`` (token and head rows may lie
+    further apart, evenly).  ``tile_seg`` / ``tile_row`` list runs of :func:`latent_row_tile` flat rows; rows
+    of other segments stay untouched."""
+    _need(q, "q", torch.bfloat16)
+    _need(out, "out", torch.bfloat16, contiguous=False)
+    _need(pages, "pages", torch.bfloat16)
+    for name, t in (("tile_seg", tile_seg), ("tile_row", tile_row), ("seg_q_start", seg_q_start),
+                    ("seg_pos0", seg_pos0), ("block_table", block_table)):
+        _need(t, name, torch.int32)
+    T, H, d = q.shape
+    if H != num_heads or pages.dim() != 4 or pages.shape[1] != 1 or pages.shape[3] != d \
+            or out.shape != (T, H, rank) or out.stride(2) != 1 or (T > 1 and out.stride(0) != H * out.stride(1)) \
+            or not attn_latent_takes(q.dtype, d, rank):
+        raise KernelError("attn_latent: shapes do not match")
+    mt = latent_row_tile(H) // 16
+    lib = build.load("attention_latent")
+    per_sm = lib.ft_attn_latent_ctas_per_sm(d, mt)
+    if per_sm == 0:
+        raise KernelError(f"attn_latent: rows of {d} values do not fit shared memory")
+    tiles = tile_seg.numel()
+    splits, split_keys = latent_splits(tiles, max_kv_len, sm_count(q.device) * per_sm)
+    part_o = part_ml = None
+    if splits > 1:
+        part_o = workspace.get("attn.part_o", (tiles * 16 * mt, splits, rank), torch.float32)
+        part_ml = workspace.get("attn.part_ml", (tiles * 16 * mt, splits, 2), torch.float32)
+    f = _fn("attention_latent", "ft_attn_latent", "p p q p p p p p p p p q i i i i i i i i i i f")
+    _check(f(_ptr(q), _ptr(out), out.stride(1), _ptr(part_o), _ptr(part_ml), _ptr(pages), _ptr(tile_seg),
+             _ptr(tile_row), _ptr(seg_q_start), _ptr(seg_pos0), _ptr(block_table), pages.stride(0), H, d, rank,
+             pages.shape[2], block_table.shape[1], int(window or 0), tiles, mt, splits, split_keys, float(scale),
+             _stream()), "attn_latent")
+    if splits > 1:
+        global LAUNCHES
+        LAUNCHES += 1
+
+
+def latent_gather(pages: torch.Tensor, dst: torch.Tensor, seg: torch.Tensor, key0: torch.Tensor,
+                  row0: torch.Tensor, seg_kv_len: torch.Tensor, seg_pos0: torch.Tensor, block_table: torch.Tensor,
+                  window: Optional[int] = None) -> None:
+    """Blocks of 64 cached rows into plain rows: block b holds keys ``key0[b] ..`` of segment ``seg[b]`` and
+    goes to rows ``row0[b] ..`` of ``dst``; keys past the segment's last, and before the first its first token
+    sees, become zeros."""
+    _need(pages, "pages", torch.bfloat16)
+    _need(dst, "dst", torch.bfloat16)
+    for name, t in (("seg", seg), ("key0", key0), ("row0", row0), ("seg_kv_len", seg_kv_len),
+                    ("seg_pos0", seg_pos0), ("block_table", block_table)):
+        _need(t, name, torch.int32)
+    if pages.dim() != 4 or pages.shape[1] != 1 or dst.shape[1] != pages.shape[3] or dst.shape[0] < 64 * seg.numel():
+        raise KernelError("latent_gather: shapes do not match")
+    f = _fn("attention_prefill_mha", "ft_latent_gather", "p p p p p p p p q i i i i i")
+    _check(f(_ptr(pages), _ptr(dst), _ptr(seg), _ptr(key0), _ptr(row0), _ptr(seg_kv_len), _ptr(seg_pos0),
+             _ptr(block_table), pages.stride(0), pages.shape[3], pages.shape[2], block_table.shape[1],
+             int(window or 0), seg.numel(), _stream()),
+           "latent_gather")
+
+
+MHA_QUERY_TILE = 128
+
+
+def attn_prefill_mha_takes(dtype: torch.dtype, dk: int, rot: int, dv: int) -> bool:
+    """Head sizes the plain-row prompt attention takes (bfloat16, multiples of 8)."""
+    return (dtype == torch.bfloat16 and dk > 0 and dk % 8 == 0 and rot % 8 == 0 and dv % 8 == 0 and 0 < dv <= 128
+            and -(-dk // 64) + -(-rot // 64) <= 4)
+
+
+def attn_prefill_mha(q: torch.Tensor, keys: torch.Tensor, shared_keys: Optional[torch.Tensor], values: torch.Tensor,
+                     out: torch.Tensor, tile_seg: torch.Tensor, tile_q0: torch.Tensor, tile_row0: torch.Tensor,
+                     seg_q_start: torch.Tensor, seg_pos0: torch.Tensor, num_heads: int, dk: int, rot: int, dv: int,
+                     scale: float, window: Optional[int] = None) -> None:
+    """Causal prompt attention over plain rows on tcgen05.  ``q`` rows are ``heads`` times ``[dk | rot]``;
+    ``keys`` ``[rows, heads, dk]`` and ``values`` ``[rows, heads, dv]`` (views of one matrix), ``shared_keys`` ``[rows, rot]``
+    (None when ``rot`` is 0); ``out`` ``[T, heads * dv]``.  ``tile_row0`` is the plain row of the tile's segment's key 0."""
+    for name, t in (("q", q), ("keys", keys), ("values", values)):
+        _need(t, name, torch.bfloat16, contiguous=False)
+    _need(out, "out", torch.bfloat16)
+    for name, t in (("tile_seg", tile_seg), ("tile_q0", tile_q0), ("tile_row0", tile_row0),
+                    ("seg_q_start", seg_q_start), ("seg_pos0", seg_pos0)):
+        _need(t, name, torch.int32)
+    T, H, rows = q.shape[0], num_heads, keys.shape[0]
+    if q.shape[1] != H * (dk + rot) or q.stride(1) != 1 or keys.shape != (rows, H, dk) or values.shape != (rows, H, dv) \
+            or keys.stride(2) != 1 or values.stride(2) != 1 or out.shape != (T, H * dv) \
+            or not attn_prefill_mha_takes(q.dtype, dk, rot, dv):
+        raise KernelError("attn_prefill_mha: shapes do not match")
+    if rot:
+        _need(shared_keys, "shared_keys", torch.bfloat16, contiguous=False)
+        if shared_keys.shape != (rows, rot) or shared_keys.stride(1) != 1:
+            raise KernelError("attn_prefill_mha: one shared key row per plain row")
+    lib = build.load("attention_prefill_mha")
+
+    def mapped(kind, t, n_rows, cols, heads, row_stride, head_stride, box):
+        def make(dst):
+            f = lib.ft_mha_map
+            f.argtypes = [ctypes.c_void_p, ctypes.c_void_p] + [ctypes.c_longlong] * 5 + [ctypes.c_int]
+            f.restype = ctypes.c_int
+            return f(dst, t.data_ptr(), n_rows, cols, heads, row_stride, head_stride, box)
+        return ctypes.cast(_attn_tc_map(kind, (t.data_ptr(), n_rows, cols, heads, row_stride, head_stride, box), make),
+                           ctypes.c_void_p)
+
+    map_q = mapped("mha_q", q, T, q.shape[1], 0, q.stride(0), 0, MHA_QUERY_TILE)
+    map_k = mapped("mha_kv", keys, rows, dk, H, keys.stride(0), keys.stride(1), 64)
+    map_v = mapped("mha_kv", values, rows, dv, H, values.stride(0), values.stride(1), 64)
+    map_r = mapped("mha_r", shared_keys, rows, rot, 0, shared_keys.stride(0), 0, 64) if rot else None
+    f = _fn("attention_prefill_mha", "ft_attn_prefill_mha", "p p p p p p p p p p p i i i i i i f")
+    _check(f(map_q, map_k, map_r, map_v, _ptr(out), _ptr(tile_seg), _ptr(tile_q0), _ptr(tile_row0),
+             _ptr(seg_q_start), _ptr(seg_pos0), _ptr(tc_status(q.device)), H, dk, rot, dv, int(window or 0),
+             tile_seg.numel(), float(scale), _stream()), "attn_prefill_mha")
 
 
 # ---------------------------------------------------------------- router

@@ -737,11 +737,12 @@ rms_rows_kernel(const AT* __restrict__ x, long long ldx, const float* __restrict
 // position (dimension 2i with 2i + 1, or i with i + rot/2) and stored behind the latent: a cached
 // row is [latent | rotated key part].  The rotated part of every head's query (the last rot of its
 // dq + rot values) is turned the same way and written behind the first rank values of the head's
-// row of q_abs ([T, heads, rank + rot]), whose first rank values another product fills.
+// row of q_abs ([T, heads, rank + rot]), whose first rank values another product fills, and / or (turn_q)
+// back into its own place.
 struct LatentStoreArgs {
   const void* down;        // [T, ld_down]: latent at column 0, the key part to rotate at column rank
-  const void* q;           // [T, ld_q]: head h at column h * (dq + rot)
-  void* q_abs;             // [T, heads, rank + rot]
+  void* q;                 // [T, ld_q]: head h at column h * (dq + rot)
+  void* q_abs;             // [T, heads, rank + rot] or nullptr
   void* pages;             // [pages, 1, P, rank + rot] or nullptr
   const float* weight;     // [rank]
   const float* cos_sin;    // [positions, rot]: cos | sin
@@ -749,7 +750,7 @@ struct LatentStoreArgs {
   const int* token_seg;
   const int* block_table;  // [segments, table_width]
   long long ld_down, ld_q, page_stride;
-  int heads, dq, rank, rot, P, table_width, interleaved;
+  int heads, dq, rank, rot, P, table_width, interleaved, turn_q;
   float eps;
 };
 
@@ -761,20 +762,22 @@ __global__ void __launch_bounds__(128) latent_store_kernel(LatentStoreArgs a) {
   const int pos = a.token_pos[t];
   const int half = a.rot >> 1;
   const float* cs = a.cos_sin + (size_t)pos * a.rot;
-  auto turn = [&](const AT* src, AT* dst, int i) {       // pair i of a rotated part
+  auto turn = [&](const AT* src, AT* dst, AT* self, int i) {       // pair i of a rotated part
     const int ia = a.interleaved ? 2 * i : i, ib = a.interleaved ? 2 * i + 1 : i + half;
     const float u = to_float(src[ia]), v = to_float(src[ib]);
     const float c = cs[i], s = cs[half + i];
-    dst[ia] = from_float<AT>(u * c - v * s);
-    dst[ib] = from_float<AT>(v * c + u * s);
+    const AT x = from_float<AT>(u * c - v * s), y = from_float<AT>(v * c + u * s);
+    if (dst) { dst[ia] = x; dst[ib] = y; }
+    if (self) { self[ia] = x; self[ib] = y; }
   };
   const int width = a.rank + a.rot;
   // queries: the rotated part of every head
-  const AT* q = (const AT*)a.q + (size_t)t * a.ld_q;
-  AT* qa = (AT*)a.q_abs + (size_t)t * a.heads * width;
+  AT* q = (AT*)a.q + (size_t)t * a.ld_q;
+  AT* qa = a.q_abs ? (AT*)a.q_abs + (size_t)t * a.heads * width : nullptr;
   for (int i = threadIdx.x; i < a.heads * half; i += blockDim.x) {
     const int h = i / half, p = i - h * half;
-    turn(q + (size_t)h * (a.dq + a.rot) + a.dq, qa + (size_t)h * width + a.rank, p);
+    AT* tail = q + (size_t)h * (a.dq + a.rot) + a.dq;
+    turn(tail, qa ? qa + (size_t)h * width + a.rank : nullptr, a.turn_q ? tail : nullptr, p);
   }
   if (!a.pages) return;
   const AT* down = (const AT*)a.down + (size_t)t * a.ld_down;
@@ -788,7 +791,7 @@ __global__ void __launch_bounds__(128) latent_store_kernel(LatentStoreArgs a) {
   const float inv = 1.f / sqrtf(block_sum(sq, scratch) / (float)a.rank + a.eps);
   for (int c = threadIdx.x; c < a.rank; c += blockDim.x)
     dst[c] = from_float<AT>(to_float(down[c]) * inv * a.weight[c]);
-  for (int i = threadIdx.x; i < half; i += blockDim.x) turn(down + a.rank, dst + a.rank, i);
+  for (int i = threadIdx.x; i < half; i += blockDim.x) turn(down + a.rank, dst + a.rank, nullptr, i);
 }
 
 
@@ -1144,14 +1147,14 @@ int ft_rms_rows(const void* x, long long ldx, const float* w, void* out, long lo
   return FT_OK;
 }
 
-int ft_latent_store(const void* down, long long ld_down, const void* q, long long ld_q, void* q_abs, void* pages,
+int ft_latent_store(const void* down, long long ld_down, void* q, long long ld_q, void* q_abs, void* pages,
                     long long page_stride, const float* weight, const float* cos_sin, const int* token_pos,
                     const int* token_seg, const int* block_table, int heads, int dq, int rank, int rot, int P,
-                    int table_width, int interleaved, float eps, int dtype, int T, cudaStream_t stream) {
+                    int table_width, int interleaved, int turn_q, float eps, int dtype, int T, cudaStream_t stream) {
   if (T <= 0) return FT_OK;
   if (heads <= 0 || dq < 0 || rank <= 0 || rot < 0 || (rot & 1) || P <= 0) return FT_ERR_SHAPE;
   LatentStoreArgs a{down, q, q_abs, pages, weight, cos_sin, token_pos, token_seg, block_table, ld_down, ld_q,
-                    page_stride, heads, dq, rank, rot, P, table_width, interleaved, eps};
+                    page_stride, heads, dq, rank, rot, P, table_width, interleaved, turn_q, eps};
   FT_DISPATCH(dtype, AT, (launch_pdl(latent_store_kernel<AT>, dim3(T), dim3(128), 0, stream, a)));
   FT_LAUNCH_CHECK();
   return FT_OK;

@@ -22,6 +22,14 @@
   X(PREFILL_CLEANER, 19, "attn_prefill_tc", "the warp that zeroes stale V rows (the last V tile)") \
   X(DECODE_PRODUCER, 21, "attn_decode_tma", "the TMA producer (a free stage)")          \
   X(DECODE_CONSUMER, 22, "attn_decode_tma", "the consumer warps (a filled stage)")      \
+  X(MHA_PRODUCER, 41, "attn_prefill_mha", "the TMA producer (a free K or V stage)")     \
+  X(MHA_MMA_Q, 42, "attn_prefill_mha", "the MMA issuer (the query tile)")               \
+  X(MHA_MMA_K, 43, "attn_prefill_mha", "the MMA issuer (a K tile)")                     \
+  X(MHA_MMA_PV, 44, "attn_prefill_mha", "the MMA issuer (P or a V tile)")               \
+  X(MHA_SOFTMAX_S, 45, "attn_prefill_mha", "the softmax warps (a score tile)")          \
+  X(MHA_SOFTMAX_PV, 46, "attn_prefill_mha", "the softmax warps (the previous P.V product)") \
+  X(MHA_SOFTMAX_LAST, 47, "attn_prefill_mha", "the softmax warps (the last P.V product)") \
+  X(MHA_SMEM_BASE, 48, "attn_prefill_mha", "the launch (shared memory off its 1,024-byte boundary)") \
   X(SELFTEST_WAIT, 31, "wait_selftest", "the waiting thread (a barrier nobody arrives at)")
 
 #define FT_STATUS_ENUM_ENTRY(name, code, kernel, role) FT_ST_##name = code,

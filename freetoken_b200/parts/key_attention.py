@@ -35,6 +35,14 @@ value instead of per head::
 The cache keeps ``[c_j | rot(k_j)]`` per token, the absorbed query is ``[Wuk,i^T q_i[:dq] | rot(q_i[dq:])]``,
 and attention runs over rows of ``rank + rot_dim`` values, of which the first ``rank`` are the "values".
 
+In bfloat16, rows of other sizes than the paged kernels' (32, 64, 128) take two kernels of their own:
+single tokens and short portions the absorbed form on tensor cores over rows of any width (each cached
+row fetched once, used as key and as value); portions of :data:`EXPAND_FROM` tokens and more the expanded form - the
+context's cached rows are gathered, ``Wuk`` and ``Wuv`` applied in one product, and every head scores its own
+``dq + rot`` values on tcgen05: per query and key ``dq + rot + dv`` instead of ``2 rank + rot`` products, for
+``rank (dq + dv)`` a key once.  Both compute the same function; which one a token takes depends on the
+length of its portion, its logits do not beyond rounding.
+
 The reference's models have neither mixer; its attention layer
 (python/freetoken/models/minimax_m2/attention.py:29-84) is the pattern both follow.
 """
@@ -43,6 +51,7 @@ from __future__ import annotations
 
 from typing import Dict, List
 
+import numpy as np
 import torch
 
 from ..cache.manager import PagedKeyNeed
@@ -50,7 +59,12 @@ from ..csrc import ops
 from ..weights.spec import Cat, Init, Name, TensorSpec
 from . import linear
 from .attention import PagedSoftmaxCore
-from .base import POSITIONS, CacheView, Mixer, StepContext, register_mixer
+from .base import POSITIONS, CacheView, Mixer, StepContext, StepPlan, StepShape, register_mixer
+
+# portions of at least this many tokens make their context's keys and values (the expanded form)
+EXPAND_FROM = 64
+# largest buffer of expanded keys and values; contexts that do not fit stay with the absorbed form
+EXPAND_BYTES = 1 << 30
 
 
 def _both_planes(pages: torch.Tensor) -> torch.Tensor:
@@ -167,7 +181,7 @@ class LatentAttention(PagedSoftmaxCore, Mixer):
             if self.position.rotary_dim != self.rot:
                 raise ValueError(f"latent_attention: the position part turns {self.position.rotary_dim} "
                                  f"dimensions, the rotated key part has {self.rot}")
-        self.full = bool(self.rot or self.q_rank or self.gate_per == "element")
+        self.full = bool(self.rot or self.q_rank or self.gate_per == "element" or not self.gated)
         if self.d > 1024:
             raise ValueError(f"latent rank plus rotated part {self.d} exceeds what the attention kernels take (1024)")
         names = p["names"]
@@ -175,6 +189,58 @@ class LatentAttention(PagedSoftmaxCore, Mixer):
         self.n = {k: f"{scope}.{v}" for k, v in names.items()}
         self.w_in = self.w_norm = self.w_uk = self.w_uv = self.w_ukt = self.w_o = None
         self.w_qnorm = self.w_uq = None
+        self.n_up = f"{scope}.{names.get('up', 'up_kv')}"        # [Wuk ; Wuv], one matrix of the model
+        self.w_up = None
+        self.own_kernels = False           # rows the paged kernels have no size for (bind decides)
+        self.expands = False
+
+    def _takes_own_kernels(self, dtype) -> bool:
+        return (self.full and self.d not in ops.DECODE_HEAD_DIMS and self.dq % 8 == 0
+                and ops.attn_latent_takes(dtype, self.d, self.rank))
+
+    def _expands(self, dtype) -> bool:
+        return (self._takes_own_kernels(dtype) and ops.attn_prefill_mha_takes(dtype, self.dq, self.rot, self.dv)
+                and self.w_in_width() % 8 == 0)
+
+    def w_in_width(self) -> int:
+        return (self.q_rank or self.nq * (self.dq + self.rot)) + self.rank + self.rot + self._gate_width()
+
+    # ---- step metadata of the kernels of its own ----------------------------------------
+    def step_plan_key(self):
+        if not self.own_kernels:
+            return super().step_plan_key()
+        return ("latent_attention", self.nq, self.dq + self.dv, self.window, self.expands)
+
+    def plan_step(self, shape: StepShape) -> StepPlan:
+        """Which segments take which form, the row tiles of the absorbed one, the query tiles, context
+        blocks and plain rows of the expanded one."""
+        if not self.own_kernels:
+            return super().plan_step(shape)
+        rt = ops.latent_row_tile(self.nq)
+        room = EXPAND_BYTES // (2 * self.nq * (self.dq + self.dv)) // 64 * 64
+        flat, tiles, blocks = [], [], []
+        rows, flat_kv, first, last = 0, 0, None, 0
+        for i, s in enumerate(shape.segments):
+            base = max(0, s.pos0 - self.window + 1) // 64 * 64 if self.window else 0
+            context = -(-(s.pos0 + s.n - base) // 64) * 64
+            if self.expands and s.n >= EXPAND_FROM and rows + context <= room:
+                tiles += [(i, q0, rows - base) for q0 in range(0, s.n, ops.MHA_QUERY_TILE)]
+                blocks += [(i, base + k, rows + k) for k in range(0, context, 64)]
+                rows += context
+                continue
+            flat += [(i, r) for r in range(0, s.n * self.nq, rt)]
+            flat_kv = max(flat_kv, s.pos0 + s.n)
+            first, last = s.q_start if first is None else first, s.q_start + s.n
+        if shape.max_q_len == 1:           # whole block-table rows: a captured graph stays put while contexts grow
+            flat_kv = shape.table_width * shape.page_size
+        arrays = {}
+        for names, items in ((("flat_seg", "flat_row"), flat), (("x_seg", "x_q0", "x_row0"), tiles),
+                             (("g_seg", "g_key0", "g_row0"), blocks)):
+            table = np.asarray(items, dtype=np.int32).reshape(-1, len(names))
+            for c, name in enumerate(names):
+                arrays[name] = np.ascontiguousarray(table[:, c])
+        return StepPlan(arrays=arrays, host={"flat": len(flat), "flat_kv": flat_kv, "flat_tokens": (first or 0, last),
+                                             "expanded": len(tiles), "rows": rows})
 
     def children(self):
         return [self.position] if self.position is not None else []
@@ -200,8 +266,8 @@ class LatentAttention(PagedSoftmaxCore, Mixer):
         specs = [
             TensorSpec(self.n["in"], (sum(piece.shape[0] for piece in pieces), W), sources=(Cat(tuple(pieces), 0),)),
             TensorSpec(self.n["latent_norm"], (R,), role="small32", init=Init(mean=1.0, std=0.0), tag="norm"),
-            TensorSpec(self.n["up_k"], (H * self.dq, R)),
-            TensorSpec(self.n["up_v"], (H * self.dv, R)),
+            TensorSpec(self.n_up, (H * (self.dq + self.dv), R), sources=(Cat((
+                Name(self.n["up_k"], (H * self.dq, R)), Name(self.n["up_v"], (H * self.dv, R))), 0),)),
             TensorSpec(self.n["o"], (W, H * self.dv), tag="residual_out"),
         ]
         if self.q_rank:
@@ -214,8 +280,10 @@ class LatentAttention(PagedSoftmaxCore, Mixer):
         H, R = self.nq, self.rank
         self.w_in = tensors[self.n["in"]]
         self.w_norm = tensors[self.n["latent_norm"]]
-        self.w_uk = tensors[self.n["up_k"]].view(H, self.dq, R)      # [head][dq, R]
-        self.w_uv = tensors[self.n["up_v"]].view(H, self.dv, R)      # [head][dv, R]
+        self.w_up = tensors[self.n_up]
+        self.w_uk = self.w_up[:H * self.dq].view(H, self.dq, R)      # [head][dq, R]
+        self.w_uv = self.w_up[H * self.dq:].view(H, self.dv, R)      # [head][dv, R]
+        self.own_kernels, self.expands = self._takes_own_kernels(dtype), self._expands(dtype)
         # the CUDA-core product wants [N, K] rows: Wuk^T per head
         self.w_ukt = self.w_uk.transpose(1, 2).contiguous() if dtype == torch.float32 else None
         self.w_o = tensors[self.n["o"]]
@@ -224,7 +292,53 @@ class LatentAttention(PagedSoftmaxCore, Mixer):
             self.w_uq = tensors[self.n["q_up"]]
 
     def libraries(self, dtype) -> List[str]:
+        if self._takes_own_kernels(dtype):
+            return (["rowwise", "attention_latent"] + (["attention_prefill_mha"] if self._expands(dtype) else [])
+                    + linear.libraries(dtype))
         return ["rowwise"] + self.attention_libraries(dtype) + linear.libraries(dtype)
+
+    def _attend_own(self, ctx: StepContext, z, q, at: int, cache: CacheView, table) -> torch.Tensor:
+        """Cache rows, then both forms of the attention, each on its segments; the heads' values ``[T, H * dv]``."""
+        T, ws = z.shape[0], ctx.workspace
+        H, R, dq, dv, rot, d = self.nq, self.rank, self.dq, self.dv, self.rot, self.d
+        plan = ctx.plan(self)
+        host, lists = plan.host, plan.tensors
+        q_abs = ws.get("lattn.q", (T, H, d), ctx.dtype) if host["flat"] else None
+        cos_sin = self.position.table(ctx.device, ctx.max_positions) if rot else None
+        ops.latent_store(z[:, at:at + R + rot], q, q_abs, cache.pages if cache.writes else None, self.w_norm,
+                         cos_sin, ctx.token_pos, ctx.token_seg, table, heads=H, q_dim=dq, rank=R, rot=rot,
+                         interleaved=bool(rot and self.position.interleaved), eps=self.eps,
+                         turn_q=host["expanded"] > 0)
+        y = ws.get("lattn.v", (T, H * dv), ctx.dtype)
+        if host["flat"]:
+            # the tokens from the first to the last absorbed segment; whatever lies between is overwritten below
+            t0, t1 = host["flat_tokens"]
+            q_heads = q[t0:t1].unflatten(1, (H, dq + rot))[:, :, :dq]
+            torch.bmm(q_heads.transpose(0, 1), self.w_uk, out=q_abs[t0:t1, :, :R].transpose(0, 1))
+            o = ws.get("lattn.o", (T, H, R), ctx.dtype)
+            ops.attn_latent(q_abs, o, cache.pages, lists["flat_seg"], lists["flat_row"], ctx.seg_q_start,
+                            ctx.seg_pos0, table, H, R, self.scale, self.window, host["flat_kv"], ws)
+            torch.bmm(o[t0:t1].transpose(0, 1), self.w_uv.transpose(1, 2),
+                      out=y.view(T, H, dv)[t0:t1].transpose(0, 1))
+        if host["expanded"]:
+            rows = host["rows"]
+            plain = ws.get("lattn.rows", (rows, d), ctx.dtype)
+            ops.latent_gather(cache.pages, plain, lists["g_seg"], lists["g_key0"], lists["g_row0"], ctx.seg_kv_len,
+                              ctx.seg_pos0, table, self.window)
+            made = ws.get("lattn.kv", (rows, H * (dq + dv)), ctx.dtype)
+            torch.matmul(plain[:, :R], self.w_up.t(), out=made)
+            ops.attn_prefill_mha(q, made[:, :H * dq].unflatten(1, (H, dq)), plain[:, R:] if rot else None,
+                                 made[:, H * dq:].unflatten(1, (H, dv)), y, lists["x_seg"], lists["x_q0"],
+                                 lists["x_row0"], ctx.seg_q_start, ctx.seg_pos0, H, dq, rot, dv, self.scale,
+                                 self.window)
+        return y
+
+    def _gate(self, y, z, at: int) -> None:
+        gate = z[:, at + self.d:]
+        if self.gate_per == "head":
+            ops.gate_heads(y, gate, self.nq, self.dv)
+        else:
+            ops.gate_heads(y, gate, self.nq * self.dv, 1)
 
     def _forward_full(self, ctx: StepContext, x: torch.Tensor, cache: CacheView, out=None) -> torch.Tensor:
         """The fuller form: a query latent, a rotated key part, a window, a gate per value."""
@@ -240,6 +354,11 @@ class LatentAttention(PagedSoftmaxCore, Mixer):
         else:
             q, at = z[:, :q_width], q_width
         table = ctx.block_tables[cache.block_table_index]
+        if self.own_kernels:
+            y = self._attend_own(ctx, z, q, at, cache, table)
+            if self.gated:
+                self._gate(y, z, at)
+            return linear.linear(y, self.w_o, ws.get("lattn.y", (T, self.hidden), ctx.dtype) if out is None else out)
         q_abs = ws.get("lattn.q", (T, H, d), ctx.dtype)
         cos_sin = self.position.table(ctx.device, ctx.max_positions) if rot else None
         ops.latent_store(z[:, at:at + R + rot], q, q_abs, cache.pages if cache.writes else None, self.w_norm,
@@ -262,11 +381,7 @@ class LatentAttention(PagedSoftmaxCore, Mixer):
         else:
             torch.bmm(o_latent.transpose(0, 1), self.w_uv.transpose(1, 2), out=y.view(T, H, dv).transpose(0, 1))
         if self.gated:
-            gate = z[:, at + R + rot:]
-            if self.gate_per == "head":
-                ops.gate_heads(y, gate, H, dv)
-            else:
-                ops.gate_heads(y, gate, H * dv, 1)
+            self._gate(y, z, at)
         if out is None:
             out = ws.get("lattn.y", (T, self.hidden), ctx.dtype)
         return linear.linear(y, self.w_o, out)
