@@ -8,7 +8,9 @@ engine is single-GPU: for ``--gpus N`` with N > 1 it says so and exits with 2.
 MiniMax-M3 decoder at equal size (freetoken_b200/design_bench.py); ``--design tonapel`` does the
 same for the Tonapel decoder (freetoken_b200/tonapel_bench.py), ``--design nirelix`` runs the Nirelix
 decoder beside the Tonapel decoder at equal size (freetoken_b200/nirelix_bench.py), ``--design mezapel``
-the Mezapel decoder beside the MiniMax-M3 decoder at equal size (freetoken_b200/mezapel_bench.py).
+the Mezapel decoder beside the MiniMax-M3 decoder at equal size (freetoken_b200/mezapel_bench.py),
+``--design dizatar`` the Dizatar decoder beside a Nirelix decoder of latent-attention layers at equal size
+(freetoken_b200/dizatar_bench.py).
 """
 import os
 import sys

@@ -70,13 +70,18 @@ __global__ void __launch_bounds__(LT_THREADS) attn_latent_kernel(LatentAttnArgs 
   const int ntiles = k_end > k_lo ? (k_end - k_begin + LT_KEYS - 1) / LT_KEYS : 0;
   const int chunks = a.d >> 3;
 
-  auto load_tile = [&](int tile, int stage) {
-    const int j0 = k_begin + tile * LT_KEYS;
-    __nv_bfloat16* dst = sK + (size_t)stage * LT_KEYS * ld;
-    for (int r = warp; r < LT_KEYS; r += LT_THREADS / 32) {
-      const int j = min(max(j0 + r, k_lo), pos_last);   // rows outside repeat a valid key (masked later)
-      const __nv_bfloat16* src = a.pages + (size_t)table[j / a.P] * a.page_stride + (size_t)(j % a.P) * a.d;
-      for (int c = lane; c < chunks; c += 32) cp_async16(dst + r * ld + c * 8, src + c * 8);
+  // A warp fetches rows warp, warp + 8, ... of a tile.  Lanes 0..7 look their row's place up (all at once);
+  // rows outside the visible keys repeat a valid one (masked later).
+  auto locate = [&](int tile) -> const __nv_bfloat16* {
+    const int j = min(max(k_begin + tile * LT_KEYS + warp + 8 * (lane & 7), k_lo), pos_last);
+    return a.pages + (size_t)table[j / a.P] * a.page_stride + (size_t)(j % a.P) * a.d;
+  };
+  auto load_tile = [&](const __nv_bfloat16* mine, int stage) {
+    __nv_bfloat16* dst = sK + (size_t)stage * LT_KEYS * ld + warp * ld;
+#pragma unroll
+    for (int i = 0; i < LT_KEYS / 8; ++i) {
+      const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(__shfl_sync(0xffffffffu, (unsigned long long)mine, i));
+      for (int c = lane; c < chunks; c += 32) cp_async16(dst + i * 8 * ld + c * 8, src + c * 8);
     }
   };
 
@@ -85,9 +90,10 @@ __global__ void __launch_bounds__(LT_THREADS) attn_latent_kernel(LatentAttnArgs 
     for (int r = tid; r < RT + a.stages * LT_KEYS; r += LT_THREADS)
       *reinterpret_cast<uint4*>((r < RT ? sQ + r * ld : sK + (size_t)(r - RT) * ld) + a.d) = make_uint4(0u, 0u, 0u, 0u);
   for (int s = 0; s < a.stages - 1; ++s) {
-    if (s < ntiles) load_tile(s, s);
+    if (s < ntiles) load_tile(locate(s), s);
     cp_async_commit();
   }
+  const __nv_bfloat16* ahead = a.stages - 1 < ntiles ? locate(a.stages - 1) : nullptr;    // the next tile to fetch
   for (int r = warp; r < RT; r += LT_THREADS / 32)
     for (int c = lane; c < chunks; c += 32) {
       uint4 v = make_uint4(0u, 0u, 0u, 0u);
@@ -119,8 +125,9 @@ __global__ void __launch_bounds__(LT_THREADS) attn_latent_kernel(LatentAttnArgs 
     else cp_async_wait<0>();
     __syncthreads();                            // the tile has landed (stages > 1); everybody is done with tile - 1
     const int pre = tile + a.stages - 1;
-    if (pre < ntiles) load_tile(pre, pre % a.stages);
+    if (pre < ntiles) load_tile(ahead, pre % a.stages);
     cp_async_commit();
+    if (pre + 1 < ntiles) ahead = locate(pre + 1);
     if (a.stages == 1) {
       cp_async_wait<0>();
       __syncthreads();

@@ -340,8 +340,8 @@ __global__ void __launch_bounds__(192, 2) attn_prefill_mha_kernel(const __grid_c
   }
 }
 
-// Cached rows of d values -> plain rows.  Block b copies the 64 rows of keys key0[b] .. of segment seg[b] to
-// plain rows row0[b] ..; keys the segment does not have, and keys before the first that
+// Cached rows of d values -> plain rows.  Eight blocks (a warp per row) copy the 64 rows of keys key0[b] .. of segment
+// seg[b] to plain rows row0[b] ..; keys the segment does not have, and keys before the first that
 // its first token sees (their pages may be another request's by now), become zeros.
 __global__ void __launch_bounds__(256) latent_gather_kernel(const __nv_bfloat16* __restrict__ pages,
                                                             __nv_bfloat16* __restrict__ dst, const int* __restrict__ seg,
@@ -356,7 +356,8 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const __nv_bfloat16*
   const int* table = block_table + (size_t)s * table_width;
   const int chunks = d >> 3;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  for (int r = warp; r < MK; r += 8) {
+  {
+    const int r = blockIdx.y * 8 + warp;               // a warp per row
     const int j = k0 + r;
     const __nv_bfloat16* src = j >= lo && j < len ? pages + (size_t)table[j / P] * page_stride + (size_t)(j % P) * d : nullptr;
     for (int c = lane; c < chunks; c += 32) {
@@ -430,7 +431,7 @@ int ft_latent_gather(const void* pages, void* dst, const int* seg, const int* ke
   if (blocks <= 0) return FT_OK;
   if (d <= 0 || (d & 7) || (page_stride & 7) || ((uintptr_t)pages & 15) || ((uintptr_t)dst & 15) || P <= 0)
     return FT_ERR_SHAPE;
-  launch_pdl(latent_gather_kernel, dim3(blocks), dim3(256), 0, stream, (const __nv_bfloat16*)pages,
+  launch_pdl(latent_gather_kernel, dim3(blocks, MK / 8), dim3(256), 0, stream, (const __nv_bfloat16*)pages,
              (__nv_bfloat16*)dst, seg, key0, row0, seg_kv_len, seg_pos0, block_table, page_stride, d, P, table_width,
              window);
   FT_LAUNCH_CHECK();

@@ -309,32 +309,37 @@ __device__ __forceinline__ float branch_at(const BranchArgs& b, int t, int H, in
   if (back != 0.f) z = fmaf(back, to_float(((const AT*)b.source)[(size_t)t * H + c]), z);
   return z;
 }
+// Which slots of token t have a row (bit j), and c_t; every lane of the (whole) warp gets both.  The ids are
+// fetched by all lanes at once, so that the rows' loads wait for one load and not for one per slot.
+__device__ __forceinline__ unsigned branch_slots(const BranchArgs& b, int t, float& back) {
+  back = 0.f;
+  if (!b.ids) return b.k >= 32 ? 0xffffffffu : (1u << b.k) - 1u;
+  const int lane = threadIdx.x & 31;
+  const int id = lane < b.k ? b.ids[(size_t)t * b.k + lane] : 0;
+  const float w = lane < b.k ? b.weights[(size_t)t * b.k + lane] : 0.f;
+  back = warp_sum(lane < b.k && id >= b.experts ? w : 0.f);
+  return __ballot_sync(0xffffffffu, lane < b.k && id < b.experts);
+}
+// columns 4g .. 4g + 3 of token t's branch (k <= 32), the rows' pieces fetched four at a time
 template <typename AT>
-__device__ __forceinline__ float4 branch_at4(const BranchArgs& b, int t, int H, int gi) {
+__device__ __forceinline__ float4 branch_at4(const BranchArgs& b, int t, int H, int gi, unsigned slots, float back) {
   const AT* rows = (const AT*)b.rows + (size_t)t * b.k * H + 4 * gi;
-  float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
-  float back = 0.f;
-  for (int j = 0; j < b.k; ++j) {
-    if (b.ids && b.ids[(size_t)t * b.k + j] >= b.experts) {
-      back += b.weights[(size_t)t * b.k + j];
-      continue;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 z = zero, e = zero, h = zero;
+  if (b.extra) e = load4f((const AT*)b.extra + (size_t)t * H + 4 * gi);
+  if (back != 0.f) h = load4f((const AT*)b.source + (size_t)t * H + 4 * gi);
+  for (int j0 = 0; j0 < b.k; j0 += 4) {
+    float4 v[4];
+#pragma unroll
+    for (int u = 0; u < 4; ++u) v[u] = (j0 + u < b.k && (slots >> (j0 + u) & 1u)) ? load4f(rows + (size_t)(j0 + u) * H) : zero;
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      const float s = (b.part_scale && j0 + u < b.k) ? b.part_scale[j0 + u] : 1.f;
+      z.x = fmaf(s, v[u].x, z.x); z.y = fmaf(s, v[u].y, z.y); z.z = fmaf(s, v[u].z, z.z); z.w = fmaf(s, v[u].w, z.w);
     }
-    const float4 v = load4f(rows + (size_t)j * H);
-    if (b.part_scale) {
-      const float s = b.part_scale[j];
-      z.x = fmaf(s, v.x, z.x); z.y = fmaf(s, v.y, z.y); z.z = fmaf(s, v.z, z.z); z.w = fmaf(s, v.w, z.w);
-    } else {
-      z.x += v.x; z.y += v.y; z.z += v.z; z.w += v.w;
-    }
   }
-  if (b.extra) {
-    const float4 v = load4f((const AT*)b.extra + (size_t)t * H + 4 * gi);
-    z.x += v.x; z.y += v.y; z.z += v.z; z.w += v.w;
-  }
-  if (back != 0.f) {
-    const float4 v = load4f((const AT*)b.source + (size_t)t * H + 4 * gi);
-    z.x = fmaf(back, v.x, z.x); z.y = fmaf(back, v.y, z.y); z.z = fmaf(back, v.z, z.z); z.w = fmaf(back, v.w, z.w);
-  }
+  z.x += e.x; z.y += e.y; z.z += e.z; z.w += e.w;
+  z.x = fmaf(back, h.x, z.x); z.y = fmaf(back, h.y, z.y); z.z = fmaf(back, h.z, z.z); z.w = fmaf(back, h.w, z.w);
   return z;
 }
 
@@ -364,29 +369,33 @@ cast_rows_kernel(float* __restrict__ x, BranchArgs b, AT* __restrict__ dst, long
   }
   dst[t * ld + c] = from_float<AT>(v);
 }
+// a block per token (16-byte pieces)
 template <typename AT>
 __global__ void __launch_bounds__(256)
-cast_rows4_kernel(float* __restrict__ x, BranchArgs b, AT* __restrict__ dst, long long ld, long long n4, int groups) {
+cast_rows4_kernel(float* __restrict__ x, BranchArgs b, AT* __restrict__ dst, long long ld, int groups) {
   pdl_wait();
-  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
-  if (i >= n4) return;
-  const int t = (int)(i / groups), g = (int)(i - (long long)t * groups);
-  float4 v = load4f(x + 4 * i);
-  if (b.rows) {
-    const float4 z = branch_at4<AT>(b, t, 4 * groups, g);
-    v.x += z.x; v.y += z.y; v.z += z.z; v.w += z.w;
-    store4f(x + 4 * i, v);
+  const int t = blockIdx.x;
+  float back = 0.f;
+  const unsigned slots = b.rows ? branch_slots(b, t, back) : 0u;
+  for (int g = threadIdx.x; g < groups; g += blockDim.x) {
+    float* p = x + ((size_t)t * groups + g) * 4;
+    float4 v = load4f(p);
+    if (b.rows) {
+      const float4 z = branch_at4<AT>(b, t, 4 * groups, g, slots, back);
+      v.x += z.x; v.y += z.y; v.z += z.z; v.w += z.w;
+      store4f(p, v);
+    }
+    store4f(dst + t * ld + 4 * g, v);
   }
-  store4f(dst + t * ld + 4 * g, v);
 }
 
 // ------------------------------------------------- a branch's own norm, then the residual
 // z as above; the residual takes mult * rms(z) * (w [+1]).  With a second weight the new residual
 // row is normed once more in the same pass and leaves as the next sublayer's input; with copy_out
 // it also leaves as it is, in the activation type.  A block owns a token; z, then the new residual
-// row, stay in shared memory (VEC: registers) between the passes.  `source` may be the buffer
+// row, stay in registers (odd sizes: shared memory) between the passes.  `source` may be the buffer
 // that next_out writes: a block reads its token's row before its first sum, and writes it after.
-constexpr int NORM_ADD_KEEP = 8;   // groups of 4 elements a thread keeps between the passes
+constexpr int NORM_ADD_KEEP = 8;   // most groups of 4 elements a thread keeps between the passes
 
 struct NormAddArgs {
   BranchArgs b;
@@ -400,9 +409,11 @@ struct NormAddArgs {
   float eps, next_eps, mult;
 };
 
-// VEC: rows of up to 4 * 256 * NORM_ADD_KEEP elements, a multiple of 4, every row 16-byte (bfloat16: 8-byte)
-// aligned: each row is read once, in 16-byte pieces, and stays in registers between the passes.
-template <typename AT, bool VEC>
+// KEEP > 0: rows of up to 4 * 256 * KEEP elements, a multiple of 4, every row 16-byte (bfloat16: 8-byte)
+// aligned: each row is read once, in 16-byte pieces, and stays in registers between the passes; the branch
+// rows, the residual and both weights are fetched before the first sum, all loads in flight together.
+// KEEP = 0: any row, element by element through shared memory.
+template <typename AT, int KEEP>
 __global__ void __launch_bounds__(256) norm_add_kernel(NormAddArgs a) {
   extern __shared__ float row[];
   __shared__ float scratch[33];
@@ -415,43 +426,54 @@ __global__ void __launch_bounds__(256) norm_add_kernel(NormAddArgs a) {
   AT* copy = a.copy_out ? (AT*)a.copy_out + (size_t)t * a.copy_ld : nullptr;
   AT* o = (AT*)a.next_out + (size_t)t * H;
   float ss = 0.f, ss2 = 0.f;
-  if constexpr (VEC) {
-    float4 keep[NORM_ADD_KEEP];
+  if constexpr (KEEP > 0) {
+    float4 keep[KEEP], x0[KEEP], w[KEEP];
     const int groups = H >> 2;
+    float back;
+    const unsigned slots = branch_slots(a.b, t, back);
 #pragma unroll
-    for (int j = 0; j < NORM_ADD_KEEP; ++j) {
+    for (int j = 0; j < KEEP; ++j) {
       const int gi = threadIdx.x + j * 256;
       if (gi < groups) {
-        const float4 z = branch_at4<AT>(a.b, t, H, gi);
-        keep[j] = z;
+        x0[j] = load4f(r + 4 * gi);
+        w[j] = load4f(a.weight + 4 * gi);
+        keep[j] = branch_at4<AT>(a.b, t, H, gi, slots, back);
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+      const int gi = threadIdx.x + j * 256;
+      if (gi < groups) {
+        const float4 z = keep[j];
         ss = fmaf(z.x, z.x, ss); ss = fmaf(z.y, z.y, ss); ss = fmaf(z.z, z.z, ss); ss = fmaf(z.w, z.w, ss);
       }
     }
     ss = block_sum(ss, scratch);
     const float inv = 1.0f / sqrtf(ss / (float)H + a.eps);
 #pragma unroll
-    for (int j = 0; j < NORM_ADD_KEEP; ++j) {
+    for (int j = 0; j < KEEP; ++j) {
       const int gi = threadIdx.x + j * 256;
       if (gi < groups) {
-        const float4 w = load4f(a.weight + 4 * gi), x0 = load4f(r + 4 * gi), z = keep[j];
-        const float4 x = make_float4(x0.x + mult * (z.x * inv * (w.x + one)), x0.y + mult * (z.y * inv * (w.y + one)),
-                                     x0.z + mult * (z.z * inv * (w.z + one)), x0.w + mult * (z.w * inv * (w.w + one)));
+        const float4 z = keep[j];
+        const float4 x = make_float4(x0[j].x + mult * (z.x * inv * (w[j].x + one)), x0[j].y + mult * (z.y * inv * (w[j].y + one)),
+                                     x0[j].z + mult * (z.z * inv * (w[j].z + one)), x0[j].w + mult * (z.w * inv * (w[j].w + one)));
         store4f(r + 4 * gi, x);
         if (copy) store4f(copy + 4 * gi, x);
         keep[j] = x;
         ss2 = fmaf(x.x, x.x, ss2); ss2 = fmaf(x.y, x.y, ss2); ss2 = fmaf(x.z, x.z, ss2); ss2 = fmaf(x.w, x.w, ss2);
+        if (a.next_weight) w[j] = load4f(a.next_weight + 4 * gi);
       }
     }
     if (!a.next_weight) return;
     ss2 = block_sum(ss2, scratch);
     const float inv2 = 1.0f / sqrtf(ss2 / (float)H + a.next_eps);
 #pragma unroll
-    for (int j = 0; j < NORM_ADD_KEEP; ++j) {
+    for (int j = 0; j < KEEP; ++j) {
       const int gi = threadIdx.x + j * 256;
       if (gi < groups) {
-        const float4 w = load4f(a.next_weight + 4 * gi), x = keep[j];
-        store4f(o + 4 * gi, make_float4(x.x * inv2 * (w.x + one2), x.y * inv2 * (w.y + one2), x.z * inv2 * (w.z + one2),
-                                        x.w * inv2 * (w.w + one2)));
+        const float4 x = keep[j];
+        store4f(o + 4 * gi, make_float4(x.x * inv2 * (w[j].x + one2), x.y * inv2 * (w[j].y + one2),
+                                        x.z * inv2 * (w[j].z + one2), x.w * inv2 * (w[j].w + one2)));
       }
     }
   } else {
@@ -526,6 +548,31 @@ glu_rows_kernel(const AT* __restrict__ gu, AT* __restrict__ mid, long long n, in
     v = act_apply(gate, kind) * up;
   }
   mid[i] = from_float<AT>(v);
+}
+
+// the same in 16-byte pieces (bfloat16, I a multiple of 8)
+__global__ void __launch_bounds__(256)
+glu_rows8_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfloat16* __restrict__ mid, long long n8, int I8, int kind,
+                 float alpha, float limit) {
+  pdl_wait();
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n8) return;
+  const long long t = i / I8;
+  const int c = (int)(i - t * I8) * 8;
+  const __nv_bfloat16* row = gu + (size_t)t * 16 * I8;
+  float gate[8], up[8], v[8];
+  unpack8(*reinterpret_cast<const uint4*>(row + c), gate);
+  unpack8(*reinterpret_cast<const uint4*>(row + 8 * I8 + c), up);
+#pragma unroll
+  for (int j = 0; j < 8; ++j) {
+    if (kind == 3) {
+      const float g = fminf(gate[j], limit), u = fminf(fmaxf(up[j], -limit), limit);
+      v[j] = g / (1.f + expf(-alpha * g)) * (u + 1.f);
+    } else {
+      v[j] = act_apply(gate[j], kind) * up[j];
+    }
+  }
+  *reinterpret_cast<uint4*>(mid + 8 * i) = pack8(v);
 }
 
 // ------------------------------------------------- several residual streams (hyper-connections)
@@ -1023,11 +1070,15 @@ int ft_norm_add(const void* branch, int k, const float* part_scale, const int* i
                    !((uintptr_t)residual & 15) && !((uintptr_t)next_weight & 15) && !((uintptr_t)next_out & 15) &&
                    !((uintptr_t)source & 15) && !((uintptr_t)extra & 15) && !((uintptr_t)copy_out & 15) &&
                    !(copy_ld & 3);
-  if (vec) {
-    FT_DISPATCH(dtype, AT, (launch_pdl(norm_add_kernel<AT, true>, dim3(T), dim3(256), 0, stream, a)));
+  if (vec && k <= 32) {
+    const dim3 g(T), th(256);
+    if (H <= 1024) { FT_DISPATCH(dtype, AT, (launch_pdl(norm_add_kernel<AT, 1>, g, th, 0, stream, a))); }
+    else if (H <= 2048) { FT_DISPATCH(dtype, AT, (launch_pdl(norm_add_kernel<AT, 2>, g, th, 0, stream, a))); }
+    else if (H <= 4096) { FT_DISPATCH(dtype, AT, (launch_pdl(norm_add_kernel<AT, 4>, g, th, 0, stream, a))); }
+    else { FT_DISPATCH(dtype, AT, (launch_pdl(norm_add_kernel<AT, NORM_ADD_KEEP>, g, th, 0, stream, a))); }
   } else {
     FT_DISPATCH(dtype, AT,
-                (launch_pdl(norm_add_kernel<AT, false>, dim3(T), dim3(256), (size_t)H * sizeof(float), stream, a)));
+                (launch_pdl(norm_add_kernel<AT, 0>, dim3(T), dim3(256), (size_t)H * sizeof(float), stream, a)));
   }
   FT_LAUNCH_CHECK();
   return FT_OK;
@@ -1059,10 +1110,9 @@ int ft_cast_rows(float* x, const void* branch, int k, const int* ids, const floa
   const long long n = (long long)T * H;
   const int groups = H / 4;
   if (!(H & 3) && !(ld & 3) && !((uintptr_t)x & 15) && !((uintptr_t)dst & 15) && !((uintptr_t)branch & 15) &&
-      !((uintptr_t)source & 15) && !((uintptr_t)extra & 15)) {
+      !((uintptr_t)source & 15) && !((uintptr_t)extra & 15) && k <= 32) {
     FT_DISPATCH(dtype, AT,
-                (launch_pdl(cast_rows4_kernel<AT>, dim3((unsigned)((n / 4 + 255) / 256)), dim3(256), 0, stream, x, b,
-                            (AT*)dst, ld, n / 4, groups)));
+                (launch_pdl(cast_rows4_kernel<AT>, dim3(T), dim3(256), 0, stream, x, b, (AT*)dst, ld, groups)));
   } else {
     FT_DISPATCH(dtype, AT,
                 (launch_pdl(cast_rows_kernel<AT>, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, x, b,
@@ -1098,6 +1148,12 @@ int ft_glu_rows(const void* gu, void* mid, int T, int I, int kind, float alpha, 
   if (T <= 0 || I <= 0) return FT_OK;
   if (kind < 0 || kind > 3) return FT_ERR_SHAPE;
   const long long n = (long long)T * I;
+  if (dtype == FT_DTYPE_BF16 && !(I & 7) && !((uintptr_t)gu & 15) && !((uintptr_t)mid & 15)) {
+    launch_pdl(glu_rows8_kernel, dim3((unsigned)((n / 8 + 255) / 256)), dim3(256), 0, stream, (const __nv_bfloat16*)gu,
+               (__nv_bfloat16*)mid, n / 8, I / 8, kind, alpha, limit);
+    FT_LAUNCH_CHECK();
+    return FT_OK;
+  }
   FT_DISPATCH(dtype, AT,
               (launch_pdl(glu_rows_kernel<AT>, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream,
                           (const AT*)gu, (AT*)mid, n, I, kind, alpha, limit)));
