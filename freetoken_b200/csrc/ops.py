@@ -1289,9 +1289,10 @@ def attn_latent_takes(dtype: torch.dtype, d: int, rank: int) -> bool:
     return dtype == torch.bfloat16 and d % 8 == 0 and rank % 8 == 0 and 0 < rank <= d <= 1024
 
 
-def latent_row_tile(num_heads: int) -> int:
-    """Flat query rows (token-major, then head) per CTA: 16, or 32 where a token has more heads."""
-    return 16 if num_heads <= 16 else 32
+def latent_row_tile(num_heads: int, d: int, rank: int) -> int:
+    """Flat query rows (token-major, then head) per CTA: 16, or 32 where a token has more heads (and
+    fragments and accumulators of 32 rows fit the registers)."""
+    return 16 if num_heads <= 16 or d > 576 or rank > 512 else 32
 
 
 def latent_splits(tiles: int, max_kv_len: int, slots: int) -> tuple:
@@ -1328,7 +1329,7 @@ def attn_latent(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, tile_se
             or out.shape != (T, H, rank) or out.stride(2) != 1 or (T > 1 and out.stride(0) != H * out.stride(1)) \
             or not attn_latent_takes(q.dtype, d, rank):
         raise KernelError("attn_latent: shapes do not match")
-    mt = latent_row_tile(H) // 16
+    mt = latent_row_tile(H, d, rank) // 16
     lib = build.load("attention_latent")
     per_sm = lib.ft_attn_latent_ctas_per_sm(d, mt)
     if per_sm == 0:
@@ -1339,9 +1340,10 @@ def attn_latent(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, tile_se
     if splits > 1:
         part_o = workspace.get("attn.part_o", (tiles * 16 * mt, splits, rank), torch.float32)
         part_ml = workspace.get("attn.part_ml", (tiles * 16 * mt, splits, 2), torch.float32)
-    f = _fn("attention_latent", "ft_attn_latent", "p p q p p p p p p p p q i i i i i i i i i i f")
+    f = _fn("attention_latent", "ft_attn_latent", "p p q p p p p p p p p p q i i i i i i i i i i f")
     _check(f(_ptr(q), _ptr(out), out.stride(1), _ptr(part_o), _ptr(part_ml), _ptr(pages), _ptr(tile_seg),
-             _ptr(tile_row), _ptr(seg_q_start), _ptr(seg_pos0), _ptr(block_table), pages.stride(0), H, d, rank,
+             _ptr(tile_row), _ptr(seg_q_start), _ptr(seg_pos0), _ptr(block_table), _ptr(tc_status(q.device)),
+             pages.stride(0), H, d, rank,
              pages.shape[2], block_table.shape[1], int(window or 0), tiles, mt, splits, split_keys, float(scale),
              _stream()), "attn_latent")
     if splits > 1:

@@ -30,6 +30,8 @@
   X(MHA_SOFTMAX_PV, 46, "attn_prefill_mha", "the softmax warps (the previous P.V product)") \
   X(MHA_SOFTMAX_LAST, 47, "attn_prefill_mha", "the softmax warps (the last P.V product)") \
   X(MHA_SMEM_BASE, 48, "attn_prefill_mha", "the launch (shared memory off its 1,024-byte boundary)") \
+  X(LATENT_TILE, 51, "attn_latent", "the consumer warps (a tile of cached rows)")       \
+  X(LATENT_PRODUCER, 52, "attn_latent", "the producer (a free stage)")                  \
   X(SELFTEST_WAIT, 31, "wait_selftest", "the waiting thread (a barrier nobody arrives at)")
 
 #define FT_STATUS_ENUM_ENTRY(name, code, kernel, role) FT_ST_##name = code,

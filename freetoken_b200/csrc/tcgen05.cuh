@@ -39,7 +39,9 @@ __device__ __forceinline__ unsigned long long global_ns() {
 constexpr unsigned long long FT_WAIT_LIMIT_NS = 2000000000ull;
 __device__ __forceinline__ bool mbar_wait(unsigned long long* bar, unsigned parity, volatile int* gave_up,
                                           unsigned long long limit_ns = FT_WAIT_LIMIT_NS) {
-  if (mbar_try(bar, parity)) return true;
+  // the global timer takes some hundred cycles to read: not before a few polls have failed
+  for (int i = 0; i < 64; ++i)
+    if (mbar_try(bar, parity)) return true;
   const unsigned long long start = global_ns();
   for (long long round = 0; round < (1ll << 28); ++round) {
     for (int i = 0; i < 64; ++i)

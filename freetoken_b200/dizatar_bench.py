@@ -102,7 +102,7 @@ def kernel_pairs(s: Dict[str, int], peaks: Dict[str, Any], reps: int = 10) -> Di
         pos, seg = ints([ctx - 1] * B), torch.arange(B, dtype=torch.int32, device=dev)
         table = torch.arange(1, n_pages + 1, dtype=torch.int32, device=dev).view(B, per_req)
         q_start = torch.arange(B + 1, dtype=torch.int32, device=dev)
-        rt = ops.latent_row_tile(H)
+        rt = ops.latent_row_tile(H, d, R)
         flat = [(i, r) for i in range(B) for r in range(0, H, rt)]
         fs, fr = ints([a for a, _ in flat]), ints([b for _, b in flat])
         planes = rotate(lambda: torch.randn(n_pages + 1, 1, P, d, device=dev, dtype=bf), n_pages * P * d * 2, most=4)

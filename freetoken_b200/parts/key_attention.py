@@ -209,14 +209,14 @@ class LatentAttention(PagedSoftmaxCore, Mixer):
     def step_plan_key(self):
         if not self.own_kernels:
             return super().step_plan_key()
-        return ("latent_attention", self.nq, self.dq + self.dv, self.window, self.expands)
+        return ("latent_attention", self.nq, self.dq + self.dv, self.d, self.rank, self.window, self.expands)
 
     def plan_step(self, shape: StepShape) -> StepPlan:
         """Which segments take which form, the row tiles of the absorbed one, the query tiles, context
         blocks and plain rows of the expanded one."""
         if not self.own_kernels:
             return super().plan_step(shape)
-        rt = ops.latent_row_tile(self.nq)
+        rt = ops.latent_row_tile(self.nq, self.d, self.rank)
         room = EXPAND_BYTES // (2 * self.nq * (self.dq + self.dv)) // 64 * 64
         flat, tiles, blocks = [], [], []
         rows, flat_kv, first, last = 0, 0, None, 0
