@@ -29,6 +29,8 @@ def silu(v):
 
 def rotate_halves(v, base, dims, first=0):
     """``v`` ``[T, heads, dim]``: dimension i of the first ``dims`` turns with i + dims/2."""
+    if dims == 0:
+        return v
     i = torch.arange(dims // 2, dtype=torch.float64)
     a = torch.arange(first, first + v.shape[0], dtype=torch.float64)[:, None] * base ** (-2.0 * i / dims)[None, :]
     cos, sin = a.cos().to(v.dtype)[:, None, :], a.sin().to(v.dtype)[:, None, :]
@@ -44,8 +46,9 @@ def latent_attention(h, w, p, m, eps):
     q = (h @ w[p + "q"].T).view(T, H, D + R)
     down = h @ w[p + "dkv"].T
     c = rms(down[:, :rank], eps) * w[p + "dkv.norm"]
-    k_rot = rotate_halves(down[:, rank:].reshape(T, 1, R), m["rot"]["base"], R)
-    q_rot = rotate_halves(q[..., D:], m["rot"]["base"], R)
+    base = m["rot"]["base"] if R else 1.0
+    k_rot = rotate_halves(down[:, rank:].reshape(T, 1, R), base, R)
+    q_rot = rotate_halves(q[..., D:], base, R)
     k = (c @ w[p + "uk"].T).view(T, H, D)
     v = (c @ w[p + "uv"].T).view(T, H, V)
     scores = (torch.einsum("ihd,jhd->hij", q[..., :D], k)
