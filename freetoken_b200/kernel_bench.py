@@ -12,6 +12,7 @@ Kernels: ``expert_gemv`` (decode experts, weight-streaming mma.sync kernel),
 experts on tcgen05/TMEM with TMA, 64 rows per expert; ``_busy``: 512 rows per expert), ``attn_decode`` (64 rows x 2,048 keys; ``_32k``: 8 rows x 32,768 keys; ``_one_plane``: the same rows over a cache
 whose one plane is keys and values), ``key_store`` (queries times temperature and keys to pages, 8,192 tokens), ``attn_prefill`` (mma.sync), ``attn_prefill_tc`` (tcgen05/TMEM, TMA-fed; ``_8k``: a
 8,192-token prompt),
+``attn_latent`` and ``attn_prefill_mha`` (latent attention: absorbed over rows of 512 + 64 values, expanded for a prompt),
 ``router`` (float32 router logits + top-k for a decode batch); ``*_flashinfer``: the same
 attention shapes through FlashInfer's trtllm-gen kernels (the reference's backend on
 this GPU), as a comparison point; ``peak_copy`` / ``peak_gemm``: a 1 GiB device copy and an
@@ -150,6 +151,42 @@ def attn_decode_one_plane(sets: int = 2, B: int = 64, ctx: int = 2048):
     def run(i):
         ops.attn_decode(q, out, kv[i % sets], None, B, pos, seg, table, NQ, NKV, D, D ** -0.5, None, ctx, ws)
     return run, B * ctx * NKV * D * 2, 4.0 * B * NQ * D * ctx, "hbm"
+
+
+def attn_latent(sets: int = 2, B: int = 64, ctx: int = 2048):
+    """Decode rows of 16 heads over latent rows of 512 + 64 values (absorbed form; every row is read once as
+    key and value): 64 rows x 2,048 keys."""
+    P, H_, R, d = 64, 16, 512, 576
+    width = ctx // P
+    planes = [torch.randn(B * width + 1, 1, P, d, device=DEV, dtype=torch.bfloat16) for _ in range(sets)]
+    table = (torch.randperm(B * width)[: B * width] + 1).to(torch.int32).view(B, width).to(DEV)
+    q = torch.randn(B, H_, d, device=DEV, dtype=torch.bfloat16)
+    out = torch.empty(B, H_, R, device=DEV, dtype=torch.bfloat16)
+    pos = torch.full((B,), ctx - 1, dtype=torch.int32, device=DEV)
+    seg, zero = torch.arange(B, dtype=torch.int32, device=DEV), torch.zeros(B, dtype=torch.int32, device=DEV)
+    starts = torch.arange(B + 1, dtype=torch.int32, device=DEV)
+    ws = Workspace(DEV)
+
+    def run(i):
+        ops.attn_latent(q, out, planes[i % sets], seg, zero, starts, pos, table, H_, R, d ** -0.5, None, ctx, ws)
+    return run, B * ctx * d * 2, 2.0 * B * H_ * ctx * (d + R), "hbm"
+
+
+def attn_prefill_mha(T: int = 2048):
+    """One prompt of 16 heads over made keys and values (expanded latent attention): 128 + 64 -> 128 values."""
+    H_, dk, rot, dv = 16, 128, 64, 128
+    q = torch.randn(T, H_ * (dk + rot), device=DEV, dtype=torch.bfloat16)
+    shared = torch.randn(T, rot, device=DEV, dtype=torch.bfloat16)
+    made = torch.randn(T, H_ * (dk + dv), device=DEV, dtype=torch.bfloat16)
+    out = torch.empty(T, H_ * dv, device=DEV, dtype=torch.bfloat16)
+    tile = torch.arange(0, T, ops.MHA_QUERY_TILE, dtype=torch.int32, device=DEV)
+    zero = torch.zeros_like(tile)
+    starts = torch.tensor([0, T], dtype=torch.int32, device=DEV)
+
+    def run(i):
+        ops.attn_prefill_mha(q, made[:, :H_ * dk].unflatten(1, (H_, dk)), shared, made[:, H_ * dk:].unflatten(1, (H_, dv)),
+                             out, zero, tile, zero, starts, zero[:1], H_, dk, rot, dv, (dk + rot) ** -0.5)
+    return run, 0, H_ * T * (T + 1.0) * (dk + rot + dv), "tensor"
 
 
 def key_store(sets: int = 4, T: int = 8192):
@@ -312,7 +349,7 @@ KERNELS: Dict[str, Callable[[], Tuple[Callable[[int], None], int, float, str]]] 
     "attn_decode": attn_decode, "attn_decode_one_plane": attn_decode_one_plane, "key_store": key_store,
     "attn_decode_32k": attn_decode_32k, "attn_prefill": attn_prefill, "attn_prefill_tc": attn_prefill_tc,
     "attn_prefill_8k": attn_prefill_8k, "attn_prefill_tc_8k": attn_prefill_tc_8k, "router": router,
-    "attn_prefill_tc_window": attn_prefill_tc_window,
+    "attn_prefill_tc_window": attn_prefill_tc_window, "attn_latent": attn_latent, "attn_prefill_mha": attn_prefill_mha,
     "peak_copy": peak_copy, "peak_read": peak_read, "peak_gemm": peak_gemm,
     "attn_decode_flashinfer": attn_decode_flashinfer, "attn_decode_32k_flashinfer": attn_decode_32k_flashinfer,
     "attn_prefill_flashinfer": attn_prefill_flashinfer, "attn_prefill_8k_flashinfer": attn_prefill_8k_flashinfer,
