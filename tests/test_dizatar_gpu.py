@@ -237,7 +237,7 @@ def paged_rows(segs, page, d):
     return pages.cuda(), table.cuda(), rows, ints(starts), ints([p for p, _ in segs]), ints([p + n for p, n in segs])
 
 
-ROWS = [(112, 96, 7, 64), (576, 512, 16, 64), (576, 512, 33, 16), (40, 24, 3, 4), (24, 24, 20, 8), (1024, 1000, 5, 64),
+ROWS = [(104, 88, 7, 64), (576, 512, 16, 64), (576, 512, 33, 16), (40, 24, 3, 4), (24, 24, 20, 8), (1024, 1000, 5, 64),
         (264, 256, 16, 32), (120, 56, 1, 12), (160, 152, 20, 64), (576, 568, 20, 64), (320, 264, 2, 16), (256, 200, 18, 64)]
 
 
@@ -269,7 +269,7 @@ def test_absorbed_attention_over_rows_of_any_width(d, rank, H, page):
     ops.check_tc_status("cuda:0")
 
 
-@pytest.mark.parametrize("dk,rot,dv,H,page,rank", [(64, 16, 40, 6, 64, 96), (128, 64, 128, 3, 64, 512), (24, 8, 8, 3, 4, 24),
+@pytest.mark.parametrize("dk,rot,dv,H,page,rank", [(56, 24, 40, 5, 64, 104), (128, 64, 128, 3, 64, 512), (24, 8, 8, 3, 4, 24),
                                                    (72, 0, 120, 2, 8, 40), (192, 64, 128, 4, 64, 256), (8, 40, 64, 5, 16, 16),
                                                    (16, 104, 72, 1, 12, 8)])
 def test_expanded_attention_over_gathered_rows(dk, rot, dv, H, page, rank):
@@ -498,7 +498,7 @@ def sharpen(config, state, asker, target, beta):
 
 
 @pytest.mark.parametrize("dtype", list(DTYPES))
-@pytest.mark.parametrize("heads,dim,rot,rank,page,loop", [(2, 16, 8, 20, 8, None), (3, 32, 16, 96, 64, (0, 1, 2)), (17, 24, 8, 40, 16, None),
+@pytest.mark.parametrize("heads,dim,rot,rank,page,loop", [(2, 16, 8, 20, 8, None), (3, 32, 24, 88, 64, (0, 1, 2)), (17, 24, 8, 40, 16, None),
                                                           (2, 24, 24, 520, 64, None), (2, 40, 32, 96, 64, (0, 1, 1))])
 def test_a_far_key_decides(tmp_path, heads, dim, rot, rank, page, loop, dtype):
     """The target stands once, first of all and right before, on and right after a page's or tile's border, up
