@@ -177,7 +177,18 @@ struct QkRopeArgs {
   float eps;
   int dn;                 // how many of a head's d values the norm's mean counts (the others are
                           // zeros that fill a head up to d)
+  // values blended with an earlier layer's of the same tokens: v <- (1 - l) v + l first (nullptr: not)
+  const void* v_first;    // [T, ld_first] rows: nkv heads of d_first values
+  const float* v_lambda;  // l, one number
+  long long ld_first;
+  int d_first;
 };
+
+// value i of KV head h of the earlier layer's row (zero where only this layer's heads are filled up)
+template <typename AT>
+__device__ __forceinline__ float first_value(const AT* row, int h, int i, int d_first) {
+  return i < d_first ? to_float(row[(size_t)h * d_first + i]) : 0.f;
+}
 
 template <typename AT>
 __global__ void qk_rope_store_kernel(QkRopeArgs a) {
@@ -274,14 +285,22 @@ __global__ void qk_rope_store_kernel(QkRopeArgs a) {
   if (vo) {
     for (int w = threadIdx.x; w < kn; w += blockDim.x) {
       const int h = w / a.d, i = w % a.d;
-      vo[(size_t)h * head_stride_cache + i] = v[w];
+      if (a.v_first) {
+        const float l = a.v_lambda[0];
+        const AT* f = (const AT*)a.v_first + (size_t)t * a.ld_first;
+        vo[(size_t)h * head_stride_cache + i] =
+            from_float<AT>((1.f - l) * to_float(v[w]) + l * first_value<AT>(f, h, i, a.d_first));
+      } else {
+        vo[(size_t)h * head_stride_cache + i] = v[w];
+      }
     }
   }
 }
 
-// Same work for bfloat16 rows in 16-byte pieces: head_dim % 8 == 0, NeoX
+// Same work for bfloat16 rows in 16-byte pieces: head_dim % 8 == 0; NeoX
 // pairing with rotary_dim % 16 == 0, so that a piece of 8 elements below R/2
-// pairs with the piece R/2 further on.
+// pairs with the piece R/2 further on; interleaved pairing with rotary_dim % 8
+// == 0, so that a piece holds four whole pairs.
 struct Chunk8 { float v[8]; };
 __device__ __forceinline__ Chunk8 unpack8(const uint4& raw) {
   const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
@@ -360,6 +379,20 @@ __device__ __forceinline__ void load8a(const float* p, float (&v)[8]) {
   v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
 }
 
+// 4 consecutive floats from a 16-byte aligned address; four pairs of a piece turned by their angles
+__device__ __forceinline__ void load4p(const float* p, float (&v)[4]) {
+  const float4 a = *reinterpret_cast<const float4*>(p);
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+}
+__device__ __forceinline__ void turn_pairs(Chunk8& x, const float (&c)[4], const float (&s)[4]) {
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float u = x.v[2 * i], v = x.v[2 * i + 1];
+    x.v[2 * i] = u * c[i] - v * s[i];
+    x.v[2 * i + 1] = v * c[i] + u * s[i];
+  }
+}
+
 // grid (tokens, parts): the blocks of a token split its heads between them;
 // with the per-layer norm every block sums the whole q and k rows itself (a
 // few KB from L2) so that no block waits for another.
@@ -408,7 +441,8 @@ __global__ void __launch_bounds__(256) qk_rope_store_vec_kernel(QkRopeArgs a) {
     __syncthreads();
   }
   const int pos = a.token_pos[t];
-  const int half = a.R >> 1, hc = half >> 3;      // rotary half, in pieces
+  const int half = a.R >> 1;
+  const int hc = a.interleaved ? 0 : half >> 3;   // rotary half, in pieces (halves; pairs stay inside a piece)
   const float* cs = (a.cos_sin && a.R > 0) ? a.cos_sin + (size_t)pos * a.R : nullptr;
   const float one = a.plus_one ? 1.f : 0.f;
   __nv_bfloat16* qo = (__nv_bfloat16*)a.q_out + (size_t)t * qn;
@@ -471,15 +505,21 @@ __global__ void __launch_bounds__(256) qk_rope_store_vec_kernel(QkRopeArgs a) {
         store8(dst + i0, y0);
         store8(dst + i1, y1);
       } else {
-        const int i0 = (ci + hc) * 8;               // pieces beyond the rotary span
+        const int i0 = (ci + hc) * 8;               // pieces beyond the rotary span, or of whole pairs
         const uint4 r0 = *reinterpret_cast<const uint4*>(src + i0);
-        float w0[8];
+        const bool pairs = a.interleaved && cs && i0 < a.R;
+        float w0[8], c[4], sn[4];
         if (a.norm_mode) load8a(nw + wbase + i0, w0);
+        if (pairs) {
+          load4p(cs + (i0 >> 1), c);
+          load4p(cs + half + (i0 >> 1), sn);
+        }
         Chunk8 x0 = unpack8(r0);
         if (a.norm_mode) {
 #pragma unroll
           for (int i = 0; i < 8; ++i) x0.v[i] = x0.v[i] * inv * (w0[i] + one);
         }
+        if (pairs) turn_pairs(x0, c, sn);
         store8(dst + i0, x0);
       }
       continue;
@@ -511,13 +551,19 @@ __global__ void __launch_bounds__(256) qk_rope_store_vec_kernel(QkRopeArgs a) {
       store8(dst + i0, y0);
       store8(dst + i1, y1);
     } else {
-      const int i0 = (ci + hc) * 8;               // pieces beyond the rotary span
+      const int i0 = (ci + hc) * 8;               // pieces beyond the rotary span, or of whole pairs
       Chunk8 x0 = load8(src + i0);
       if (a.norm_mode) {
         float w0[8];
         load8w(nw + wbase + i0, w0);
 #pragma unroll
         for (int i = 0; i < 8; ++i) x0.v[i] = x0.v[i] * inv * (w0[i] + one);
+      }
+      if (a.interleaved && cs && i0 < a.R) {
+        float c[4], sn[4];
+        load4p(cs + (i0 >> 1), c);
+        load4p(cs + half + (i0 >> 1), sn);
+        turn_pairs(x0, c, sn);
       }
       store8(dst + i0, x0);
     }
@@ -528,8 +574,19 @@ __global__ void __launch_bounds__(256) qk_rope_store_vec_kernel(QkRopeArgs a) {
     const int v_begin = (int)((long long)vc * part / parts), v_end = (int)((long long)vc * (part + 1) / parts);
     for (int c = v_begin + threadIdx.x; c < v_end; c += blockDim.x) {
       const int h = (c * 8) / d, i = (c * 8) % d;
-      *reinterpret_cast<uint4*>(vo + (size_t)h * head_stride_cache + i) =
-          *reinterpret_cast<const uint4*>(v + c * 8);
+      uint4 piece = *reinterpret_cast<const uint4*>(v + c * 8);
+      if (a.v_first) {                              // d_first is a multiple of 8: a piece is inside or outside
+        const float l = a.v_lambda[0];
+        Chunk8 x = unpack8(piece);
+        Chunk8 f = {};
+        if (i < a.d_first)
+          f = load8((const __nv_bfloat16*)a.v_first + (size_t)t * a.ld_first + (size_t)h * a.d_first + i);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) x.v[j] = (1.f - l) * x.v[j] + l * f.v[j];
+        store8(vo + (size_t)h * head_stride_cache + i, x);
+      } else {
+        *reinterpret_cast<uint4*>(vo + (size_t)h * head_stride_cache + i) = piece;
+      }
     }
   }
 }
@@ -668,18 +725,22 @@ int ft_qk_rope_store(const void* qkv, void* q_out, void* kv_pages, const float* 
                      const int* token_seg, const int* block_table, long long ld,
                      long long page_stride, long long kv_stride, int nq, int nkv, int d, int R,
                      int P, int table_width, int norm_mode, int plus_one, int interleaved,
-                     float eps, int dtype, int T, int norm_dim, cudaStream_t stream) {
+                     float eps, int dtype, int T, int norm_dim, const void* v_first, const float* v_lambda,
+                     long long ld_first, int d_first, cudaStream_t stream) {
   if (T <= 0) return FT_OK;
+  if (v_first && (!v_lambda || d_first <= 0 || ld_first < (long long)nkv * d_first)) return FT_ERR_SHAPE;
   if (R < 0 || R > d || (R & 1) || norm_mode < 0 || norm_mode > 2) return FT_ERR_SHAPE;
   if (norm_dim <= 0 || norm_dim > d) norm_dim = d;
   QkRopeArgs a{qkv, q_out, kv_pages, q_weight, k_weight, cos_sin, token_pos, token_seg,
                block_table, ld, page_stride, kv_stride, nq, nkv, d, R, P, table_width,
-               norm_mode, plus_one, interleaved, eps, norm_dim};
+               norm_mode, plus_one, interleaved, eps, norm_dim, v_first, v_lambda, ld_first, d_first};
   const size_t smem = (size_t)(nq + nkv) * sizeof(float);
   const bool aligned = !((uintptr_t)qkv & 15) && !((uintptr_t)q_out & 15) &&
                        !((uintptr_t)kv_pages & 15) && !(ld & 7) && !(page_stride & 7) &&
-                       !(kv_stride & 7);
-  if (dtype == FT_DTYPE_BF16 && aligned && !(d & 7) && !(R & 15) && !interleaved) {
+                       !(kv_stride & 7) &&
+                       (!v_first || (!((uintptr_t)v_first & 15) && !(ld_first & 7) && !(d_first & 7)));
+  const bool whole = interleaved ? !(R & 7) && !((uintptr_t)cos_sin & 15) : !(R & 15);
+  if (dtype == FT_DTYPE_BF16 && aligned && !(d & 7) && whole) {
     // few tokens: several blocks per token share its heads
     const int pieces = (nq + 2 * nkv) * (d >> 3);
     int parts = T >= 512 ? 1 : (pieces + 255) / 256;

@@ -19,15 +19,23 @@ namespace ft {
 __device__ __forceinline__ void select_token(const float* __restrict__ x, const float* __restrict__ bias,
                                              float* score, float* choice, int* ids_out, float* weights_out,
                                              int E, int k, int softmax_scoring, int renormalize, float scale,
-                                             int terms, int groups, int keep, int lane, int& my_id,
-                                             float& my_w) {
+                                             int terms, int groups, int keep, int group_top, float* tail, int lane,
+                                             int& my_id, float& my_w) {
   // a row holds `terms` partial logits per expert, E apart (the router weight
   // split into bfloat16 terms); they are summed in order, in float32.  A lane takes
   // experts lane, lane + 32, ...; it fetches eight of them at a time into registers
   // before it touches shared memory, so that its loads from global memory are in flight
   // together (one after the other they were most of this function's time: each waits
   // for L2)
+  // With `tail` a row has one more logit behind the experts' (per term): a gate of the token, not an
+  // expert; its sigmoid goes there.
   constexpr int EPL = 8;
+  const int ld = E + (tail ? 1 : 0);
+  if (tail && lane == 0) {
+    float z = x[E];
+    for (int p = 1; p < terms; ++p) z += x[p * ld + E];
+    *tail = 1.f / (1.f + expf(-z));
+  }
   auto load_logits = [&](int base, float (&v)[EPL]) {
 #pragma unroll
     for (int i = 0; i < EPL; ++i) {
@@ -38,7 +46,7 @@ __device__ __forceinline__ void select_token(const float* __restrict__ x, const 
 #pragma unroll
       for (int i = 0; i < EPL; ++i) {
         const int e = base + i * 32 + lane;
-        if (e < E) v[i] += x[p * E + e];
+        if (e < E) v[i] += x[p * ld + e];
       }
     }
   };
@@ -89,7 +97,7 @@ __device__ __forceinline__ void select_token(const float* __restrict__ x, const 
   __syncwarp();
   if (groups > 1) {
     // Experts form `groups` equal groups of neighbours; a group's value is the sum of its two
-    // largest choice values, and only experts of the `keep` best groups stay eligible (the
+    // largest choice values (group_top 2) or the largest (group_top 1), and only experts of the `keep` best groups stay eligible (the
     // others count as minus infinity).  Lane l owns groups l, l + 32, ...; the best group is
     // found `keep` times by a warp-wide argmax (the first of equal groups wins).
     constexpr int GPL = 8;                     // groups <= 256
@@ -107,7 +115,7 @@ __device__ __forceinline__ void select_token(const float* __restrict__ x, const 
           if (c > a) { b = a; a = c; }
           else if (c > b) b = c;
         }
-        gs[i] = per > 1 ? a + b : a;
+        gs[i] = per > 1 && group_top > 1 ? a + b : a;
       }
     }
     for (int j = 0; j < keep; ++j) {
@@ -176,7 +184,7 @@ template <int WARPS>
 __global__ void router_select_kernel(const float* __restrict__ logits, const float* __restrict__ bias,
                                      int* __restrict__ ids, float* __restrict__ weights, int T, int E,
                                      int k, int softmax_scoring, int renormalize, float scale, int terms,
-                                     int groups, int keep) {
+                                     int groups, int keep, int group_top, float* __restrict__ tail) {
   extern __shared__ float smem[];  // [WARPS][2][E]: scores, choice values
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   pdl_wait();
@@ -186,9 +194,9 @@ __global__ void router_select_kernel(const float* __restrict__ logits, const flo
   float* score = smem + (size_t)warp * 2 * E;
   int my_id;
   float my_w;
-  select_token(logits + (size_t)t * E * terms, bias, score, score + E, ids + (size_t)t * k,
-               weights + (size_t)t * k, E, k, softmax_scoring, renormalize, scale, terms, groups, keep, lane, my_id,
-               my_w);
+  select_token(logits + (size_t)t * (E + (tail ? 1 : 0)) * terms, bias, score, score + E, ids + (size_t)t * k,
+               weights + (size_t)t * k, E, k, softmax_scoring, renormalize, scale, terms, groups, keep, group_top,
+               tail ? tail + t : nullptr, lane, my_id, my_w);
   if (k <= 32 && lane < k) {
     ids[(size_t)t * k + lane] = my_id;
     weights[(size_t)t * k + lane] = my_w;
@@ -206,7 +214,8 @@ __global__ void __launch_bounds__(SMALL_WARPS * 32) route_small_kernel(
     const float* __restrict__ logits, const float* __restrict__ bias, int* __restrict__ ids,
     float* __restrict__ weights, int* __restrict__ counts, int* __restrict__ offsets,
     int* __restrict__ sorted_route, int* __restrict__ sorted_token, int* __restrict__ active, int T, int E,
-    int busy_of, int k, int softmax_scoring, int renormalize, float scale, int terms, int groups, int keep) {
+    int busy_of, int k, int softmax_scoring, int renormalize, float scale, int terms, int groups, int keep,
+    int group_top, float* __restrict__ tail) {
   extern __shared__ float smem[];  // [T][2][E] scores and choices, then ints: ids [T*k], counts [E], before [E]
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int R = T * k;
@@ -219,8 +228,9 @@ __global__ void __launch_bounds__(SMALL_WARPS * 32) route_small_kernel(
     int my_id;
     float my_w;
     float* score = smem + (size_t)warp * 2 * E;
-    select_token(logits + (size_t)warp * E * terms, bias, score, score + E, nullptr, nullptr, E, k,
-                 softmax_scoring, renormalize, scale, terms, groups, keep, lane, my_id, my_w);
+    select_token(logits + (size_t)warp * (E + (tail ? 1 : 0)) * terms, bias, score, score + E, nullptr, nullptr, E, k,
+                 softmax_scoring, renormalize, scale, terms, groups, keep, group_top, tail ? tail + warp : nullptr, lane,
+                 my_id, my_w);
     if (lane < k) {
       ids[warp * k + lane] = my_id;
       weights[warp * k + lane] = my_w;
@@ -543,9 +553,9 @@ extern "C" {
 
 int ft_router_select(const float* logits, const float* bias, int* ids, float* weights, int T,
                      int E, int k, int softmax_scoring, int renormalize, float scale, int terms,
-                     int groups, int keep, cudaStream_t stream) {
+                     int groups, int keep, int group_top, float* tail, cudaStream_t stream) {
   if (T <= 0) return FT_OK;
-  if (k <= 0 || k > E || terms < 1) return FT_ERR_SHAPE;
+  if (k <= 0 || k > E || terms < 1 || group_top < 1 || group_top > 2) return FT_ERR_SHAPE;
   if (groups < 1 || groups > 256 || E % groups || keep < 1 || keep > groups || keep * (E / groups) < k)
     return FT_ERR_SHAPE;
   constexpr int WARPS = 4;
@@ -554,7 +564,7 @@ int ft_router_select(const float* logits, const float* bias, int* ids, float* we
   if (smem > 48 * 1024)
     cudaFuncSetAttribute(router_select_kernel<WARPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   launch_pdl(router_select_kernel<WARPS>, dim3((T + WARPS - 1) / WARPS), dim3(WARPS * 32), smem, stream,
-             logits, bias, ids, weights, T, E, k, softmax_scoring, renormalize, scale, terms, groups, keep);
+             logits, bias, ids, weights, T, E, k, softmax_scoring, renormalize, scale, terms, groups, keep, group_top, tail);
   FT_LAUNCH_CHECK();
   return FT_OK;
 }
@@ -562,10 +572,12 @@ int ft_router_select(const float* logits, const float* bias, int* ids, float* we
 // router_select + moe_sort in one launch; T <= 8 tokens, k <= 32.  `busy_of` as in ft_moe_sort.
 int ft_route_small(const float* logits, const float* bias, int* ids, float* weights, int* counts,
                    int* offsets, int* sorted_route, int* sorted_token, int* active, int T, int E, int busy_of, int k,
-                   int softmax_scoring, int renormalize, float scale, int terms, int groups, int keep,
-                   cudaStream_t stream) {
+                   int softmax_scoring, int renormalize, float scale, int terms, int groups, int keep, int group_top,
+                   float* tail, cudaStream_t stream) {
   if (T <= 0) return FT_OK;
-  if (T > SMALL_WARPS || k <= 0 || k > 32 || k > E || terms < 1 || busy_of < 1 || busy_of > E) return FT_ERR_SHAPE;
+  if (T > SMALL_WARPS || k <= 0 || k > 32 || k > E || terms < 1 || busy_of < 1 || busy_of > E || group_top < 1 ||
+      group_top > 2)
+    return FT_ERR_SHAPE;
   if (groups < 1 || groups > 256 || E % groups || keep < 1 || keep > groups || keep * (E / groups) < k)
     return FT_ERR_SHAPE;
   const size_t smem = (size_t)T * 2 * E * sizeof(float) + ((size_t)T * k + 2 * (size_t)E) * sizeof(int);
@@ -574,7 +586,7 @@ int ft_route_small(const float* logits, const float* bias, int* ids, float* weig
     cudaFuncSetAttribute(route_small_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   launch_pdl(route_small_kernel, dim3(1), dim3(SMALL_WARPS * 32), smem, stream, logits, bias, ids, weights,
              counts, offsets, sorted_route, sorted_token, active, T, E, busy_of, k, softmax_scoring, renormalize, scale,
-             terms, groups, keep);
+             terms, groups, keep, group_top, tail);
   FT_LAUNCH_CHECK();
   return FT_OK;
 }

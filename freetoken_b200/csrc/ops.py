@@ -154,10 +154,13 @@ def qk_rope_store(qkv: torch.Tensor, q_out: torch.Tensor, kv_pages: Optional[tor
                   cos_sin: Optional[torch.Tensor], token_pos: torch.Tensor,
                   token_seg: torch.Tensor, block_table: torch.Tensor, num_heads: int,
                   num_kv_heads: int, head_dim: int, rotary_dim: int, norm_mode: int,
-                  plus_one: bool, interleaved: bool, eps: float, norm_dim: int = 0) -> None:
+                  plus_one: bool, interleaved: bool, eps: float, norm_dim: int = 0,
+                  value_first: Optional[torch.Tensor] = None, value_lambda: Optional[torch.Tensor] = None) -> None:
     """QK norm (0 none, 1 per layer, 2 per head), partial rotary, K/V page store.
     ``norm_dim`` (0: ``head_dim``): how many of a head's values the norm's mean counts, where
-    query and key heads were filled up with zeros to ``head_dim``.
+    query and key heads were filled up with zeros to ``head_dim``.  ``value_first`` (rows of another layer's
+    values of the same tokens, ``[T, num_kv_heads * its head size]``, rows may lie further apart) with ``value_lambda``
+    (one float32 number): the stored values are ``(1 - lambda) v + lambda first``.
 
     ``kv_pages`` is ``[2, pages, kv_heads, page_size, head_dim]`` or ``None``
     for a stop that reads another stop's cache."""
@@ -188,13 +191,21 @@ def qk_rope_store(qkv: torch.Tensor, q_out: torch.Tensor, kv_pages: Optional[tor
         _need(cos_sin, "cos_sin", torch.float32)
         if cos_sin.shape[1] != rotary_dim:
             raise KernelError("qk_rope_store: cos_sin table width differs from rotary_dim")
+    d_first = 0
+    if value_first is not None:
+        _need(value_first, "value_first", qkv.dtype, contiguous=False)
+        _need(value_lambda, "value_lambda", torch.float32)
+        d_first = value_first.shape[1] // num_kv_heads
+        if value_first.shape != (T, num_kv_heads * d_first) or value_first.stride(1) != 1 or value_lambda.numel() != 1:
+            raise KernelError("qk_rope_store: value_first must be [T, kv_heads * size] with one lambda")
     f = _fn("elementwise", "ft_qk_rope_store",
-            "p p p p p p p p p q q q i i i i i i i i i f i i i")
+            "p p p p p p p p p q q q i i i i i i i i i f i i i p p q i")
     _check(f(_ptr(qkv), _ptr(q_out), _ptr(kv_pages), _ptr(q_weight), _ptr(k_weight),
              _ptr(cos_sin) if rotary_dim else None, _ptr(token_pos), _ptr(token_seg),
              _ptr(block_table), qkv.stride(0), page_stride, kv_stride, num_heads, num_kv_heads,
              head_dim, rotary_dim, P, block_table.shape[1], norm_mode, int(plus_one),
-             int(interleaved), float(eps), code(qkv.dtype), T, int(norm_dim), _stream()), "qk_rope_store")
+             int(interleaved), float(eps), code(qkv.dtype), T, int(norm_dim), _ptr(value_first), _ptr(value_lambda),
+             value_first.stride(0) if value_first is not None else 0, d_first, _stream()), "qk_rope_store")
 
 
 def combine(parts: torch.Tensor, out: torch.Tensor, k: int) -> None:
@@ -329,11 +340,11 @@ def gate_heads(o: torch.Tensor, z: torch.Tensor, heads: int, head_dim: int) -> N
     _check(f(_ptr(o), _ptr(z), z.stride(0), heads, head_dim, code(o.dtype), T, _stream()), "gate_heads")
 
 
-ACTIVATIONS = {"relu2": 0, "gelu_tanh": 1, "silu": 2}
+ACTIVATIONS = {"relu2": 0, "gelu_tanh": 1, "silu": 2, "tanh": 4}
 
 
 def activation(x: torch.Tensor, kind: str) -> None:
-    """In place: ``relu2`` relu(x)^2, ``gelu_tanh``, ``silu``; float32 arithmetic."""
+    """In place: ``relu2`` relu(x)^2, ``gelu_tanh``, ``silu``, ``tanh``; float32 arithmetic."""
     _need(x, "x")
     if kind not in ACTIVATIONS:
         raise KernelError(f"activation: unknown kind {kind!r}")
@@ -351,38 +362,73 @@ def softcap(x: torch.Tensor, cap: float) -> None:
 
 # ------------------------------------- sandwich norms, sums of mixers, biases, gated rows
 class RoutedRows:
-    """What a routed feed-forward hands on, not added up yet: ``rows`` ``[T, k, H]``, of which slots
-    whose id (``ids`` ``[T, k]``) is ``experts`` or more were never written - such a slot hands the
-    branch's input ``source`` (``[T, H]``) back, times its weight (``weights`` ``[T, k]``) -, and ``extra``
-    (``[T, H]`` or None), one more row per token.  The value of a token is the sum of all that."""
+    """What a sublayer hands on, not added up yet: ``rows`` ``[T, k, H]`` (or ``[T, H]``; ``scale`` ``[k]`` or
+    None: a factor per partial row), of which slots whose id (``ids`` ``[T, k]``) is ``experts`` or more
+    were never written - such a slot hands the branch's input ``source`` (``[T, H]``) back, times its weight
+    (``weights`` ``[T, k]``); ``extra`` (``[T, H]`` or None), one more row per token, times ``extra_gate``
+    (float32 ``[T]`` or None: 1); and ``beside`` (``[T, m, H]`` or ``[T, H]`` or None), the rows of another
+    sublayer that read the same input, times ``beside_scale`` (float32 ``[m]`` or None: 1).  The value of a
+    token is the sum of all that, in float32."""
 
-    __slots__ = ("rows", "ids", "weights", "experts", "source", "extra")
+    __slots__ = ("rows", "ids", "weights", "experts", "source", "extra", "scale", "extra_gate", "beside",
+                 "beside_scale")
 
-    def __init__(self, rows, ids=None, weights=None, experts: int = 0, source=None, extra=None):
+    def __init__(self, rows, ids=None, weights=None, experts: int = 0, source=None, extra=None, scale=None,
+                 extra_gate=None, beside=None, beside_scale=None):
         self.rows, self.ids, self.weights, self.experts = rows, ids, weights, int(experts)
-        self.source, self.extra = source, extra
+        self.source, self.extra, self.scale, self.extra_gate = source, extra, scale, extra_gate
+        self.beside, self.beside_scale = beside, beside_scale
+
+
+class _BranchArgs(ctypes.Structure):
+    """Field by field the struct of the same name in rowwise.cu."""
+
+    _fields_ = ([(n, ctypes.c_void_p) for n in ("rows", "part_scale", "ids", "weights", "source", "extra", "extra_gate",
+                                                "beside", "beside_scale")]
+                + [(n, ctypes.c_int) for n in ("k", "experts", "kb")])
 
 
 def _branch_args(branch, T: int, H: int, name: str):
-    """``(rows tensor, k, ids, weights, experts, source, extra)`` of a branch output, checked."""
-    if not isinstance(branch, RoutedRows):
-        branch = RoutedRows(branch)
-    rows = branch.rows
+    """``(address of the kernels' view of a branch output, its element type, the object to keep alive
+    meanwhile)``, checked."""
+    b = branch if isinstance(branch, RoutedRows) else RoutedRows(branch)
+    rows = b.rows
     _need(rows, "branch")
     k = rows.shape[1] if rows.dim() == 3 else 1
     if rows.shape[0] != T or rows.shape[-1] != H:
         raise KernelError(f"{name}: shapes do not match")
-    if branch.ids is not None:
-        _need(branch.ids, "ids", torch.int32)
-        _need(branch.weights, "weights", torch.float32)
-        _need(branch.source, "source", rows.dtype)
-        if branch.ids.numel() != T * k or branch.weights.numel() != T * k or branch.source.shape != (T, H):
+    if b.scale is not None:
+        _need(b.scale, "scale", torch.float32)
+        if b.scale.numel() != k or b.ids is not None:
+            raise KernelError(f"{name}: one scale per partial row (and no ids beside scales)")
+    if b.ids is not None:
+        _need(b.ids, "ids", torch.int32)
+        _need(b.weights, "weights", torch.float32)
+        _need(b.source, "source", rows.dtype)
+        if b.ids.numel() != T * k or b.weights.numel() != T * k or b.source.shape != (T, H):
             raise KernelError(f"{name}: one id and one weight per partial row, one source row per token")
-    if branch.extra is not None:
-        _need(branch.extra, "extra", rows.dtype)
-        if branch.extra.shape != (T, H):
+    if b.extra is not None:
+        _need(b.extra, "extra", rows.dtype)
+        if b.extra.shape != (T, H):
             raise KernelError(f"{name}: one extra row per token")
-    return rows, k, branch.ids, branch.weights, branch.experts, branch.source, branch.extra
+    if b.extra_gate is not None:
+        _need(b.extra_gate, "extra_gate", torch.float32)
+        if b.extra is None or b.extra_gate.numel() != T:
+            raise KernelError(f"{name}: one gate per extra row")
+    kb = 0
+    if b.beside is not None:
+        _need(b.beside, "beside", rows.dtype)
+        kb = b.beside.shape[1] if b.beside.dim() == 3 else 1
+        if b.beside.shape[0] != T or b.beside.shape[-1] != H:
+            raise KernelError(f"{name}: the other sublayer's rows do not fit")
+    if b.beside_scale is not None:
+        _need(b.beside_scale, "beside_scale", torch.float32)
+        if b.beside_scale.numel() != kb:
+            raise KernelError(f"{name}: one scale per row of the other sublayer")
+    p = lambda t: t.data_ptr() if t is not None else None
+    args = _BranchArgs(p(rows), p(b.scale), p(b.ids), p(b.weights), p(b.source), p(b.extra), p(b.extra_gate),
+                       p(b.beside), p(b.beside_scale), k, b.experts, kb)
+    return ctypes.addressof(args), rows.dtype, args
 
 
 def norm_add(branch, residual: torch.Tensor, weight: torch.Tensor, eps: float,
@@ -397,37 +443,58 @@ def norm_add(branch, residual: torch.Tensor, weight: torch.Tensor, eps: float,
     _need(residual, "residual", torch.float32)
     _need(weight, "weight", torch.float32)
     T, H = residual.shape
-    rows, k, ids, weights, experts, source, extra = _branch_args(branch, T, H, "norm_add")
+    if part_scale is not None:
+        if isinstance(branch, RoutedRows):
+            raise KernelError("norm_add: a routed branch carries its scales itself")
+        branch = RoutedRows(branch, scale=part_scale)
+    address, dtype, _alive = _branch_args(branch, T, H, "norm_add")
     if weight.numel() != H:
         raise KernelError("norm_add: shapes do not match")
-    if part_scale is not None:
-        _need(part_scale, "part_scale", torch.float32)
-        if part_scale.numel() != k or ids is not None:
-            raise KernelError("norm_add: one scale per partial row (and no ids beside scales)")
     if next_weight is not None:
         _need(next_weight, "next_weight", torch.float32)
-        _need(next_out, "next_out", rows.dtype)
+        _need(next_out, "next_out", dtype)
         if next_out.shape != residual.shape or next_weight.numel() != H:
             raise KernelError("norm_add: the second norm's shapes do not match")
     if copy_out is not None:
-        _need(copy_out, "copy_out", rows.dtype, contiguous=False)
+        _need(copy_out, "copy_out", dtype, contiguous=False)
         if copy_out.shape != residual.shape or copy_out.stride(1) != 1:
             raise KernelError("norm_add: copy_out must be [T, H] with unit stride")
-    f = _fn("rowwise", "ft_norm_add", "p i p p p i p p p i f f p p i f p p q i i i")
-    _check(f(_ptr(rows), k, _ptr(part_scale), _ptr(ids), _ptr(weights), experts, _ptr(source), _ptr(extra),
-             _ptr(weight), int(plus_one), float(eps), float(mult), _ptr(residual), _ptr(next_weight),
+    f = _fn("rowwise", "ft_norm_add", "p p i f f p p i f p p q i i i")
+    _check(f(address, _ptr(weight), int(plus_one), float(eps), float(mult), _ptr(residual), _ptr(next_weight),
              int(next_plus_one), float(next_eps), _ptr(next_out), _ptr(copy_out),
-             copy_out.stride(0) if copy_out is not None else 0, T, H, code(rows.dtype), _stream()), "norm_add")
+             copy_out.stride(0) if copy_out is not None else 0, T, H, code(dtype), _stream()), "norm_add")
+
+
+def join_layer_norm(branch, residual: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor,
+                    bias: Optional[torch.Tensor] = None, weight2: Optional[torch.Tensor] = None, eps2: float = 0.0,
+                    out2: Optional[torch.Tensor] = None, bias2: Optional[torch.Tensor] = None) -> None:
+    """``residual += value of branch`` (``[T, H]``, ``[T, k, H]`` or :class:`RoutedRows`; None: nothing joins),
+    then ``out = (x - mean) / sqrt(variance + eps) * weight [+ bias]`` of the new rows and, with
+    ``weight2``, ``out2`` likewise: two norms of one row, its mean and variance taken once.  float32 throughout."""
+    _need(residual, "residual", torch.float32)
+    T, H = residual.shape
+    address, dtype, _alive = _branch_args(branch, T, H, "join_layer_norm") if branch is not None else (None, out.dtype, None)
+    for name, t, o, b in (("weight", weight, out, bias), ("weight2", weight2, out2, bias2)):
+        if t is None:
+            continue
+        _need(t, name, torch.float32)
+        _need(o, "out", dtype)
+        if b is not None:
+            _need(b, "bias", torch.float32)
+        if t.numel() != H or o.shape != residual.shape or (b is not None and b.numel() != H):
+            raise KernelError("join_layer_norm: shapes do not match")
+    f = _fn("rowwise", "ft_join_layer_norm", "p p p p f p p p f p i i i")
+    _check(f(address, _ptr(residual), _ptr(weight), _ptr(bias), float(eps), _ptr(out), _ptr(weight2), _ptr(bias2),
+             float(eps2), _ptr(out2), T, H, code(dtype), _stream()), "join_layer_norm")
 
 
 def branch_sum(branch, out: torch.Tensor) -> None:
     """out[t, :] = the value of token t of ``branch`` (``[T, k, H]`` or :class:`RoutedRows`), summed in float32."""
     T, H = out.shape
-    rows, k, ids, weights, experts, source, extra = _branch_args(branch, T, H, "branch_sum")
-    _need(out, "out", rows.dtype)
-    f = _fn("rowwise", "ft_branch_sum", "p i p p i p p p i i i")
-    _check(f(_ptr(rows), k, _ptr(ids), _ptr(weights), experts, _ptr(source), _ptr(extra), _ptr(out), T, H,
-             code(rows.dtype), _stream()), "branch_sum")
+    address, dtype, _alive = _branch_args(branch, T, H, "branch_sum")
+    _need(out, "out", dtype)
+    f = _fn("rowwise", "ft_branch_sum", "p p i i i")
+    _check(f(address, _ptr(out), T, H, code(dtype), _stream()), "branch_sum")
 
 
 def cast_rows(x: torch.Tensor, dst: torch.Tensor, branch=None) -> None:
@@ -438,14 +505,13 @@ def cast_rows(x: torch.Tensor, dst: torch.Tensor, branch=None) -> None:
     if dst.shape != x.shape or dst.dim() != 2 or dst.stride(1) != 1:
         raise KernelError("cast_rows: dst must be [T, H] with unit stride")
     T, H = x.shape
-    rows, k, ids, weights, experts, source, extra = (None, 0, None, None, 0, None, None)
+    address, _alive = None, None
     if branch is not None:
-        rows, k, ids, weights, experts, source, extra = _branch_args(branch, T, H, "cast_rows")
-        if rows.dtype != dst.dtype:
+        address, dtype, _alive = _branch_args(branch, T, H, "cast_rows")
+        if dtype != dst.dtype:
             raise KernelError("cast_rows: the branch and dst must have one element type")
-    f = _fn("rowwise", "ft_cast_rows", "p p i p p i p p p q i i i")
-    _check(f(_ptr(x), _ptr(rows), k, _ptr(ids), _ptr(weights), experts, _ptr(source), _ptr(extra), _ptr(dst),
-             dst.stride(0), T, H, code(dst.dtype), _stream()), "cast_rows")
+    f = _fn("rowwise", "ft_cast_rows", "p p p q i i i")
+    _check(f(_ptr(x), address, _ptr(dst), dst.stride(0), T, H, code(dst.dtype), _stream()), "cast_rows")
 
 
 def scaled_sum(parts: torch.Tensor, scale: torch.Tensor, out: torch.Tensor) -> None:
@@ -470,7 +536,7 @@ def bias_add(x: torch.Tensor, bias: torch.Tensor) -> None:
     _check(f(_ptr(x), x.stride(0), _ptr(bias), x.shape[0], x.shape[1], code(x.dtype), _stream()), "bias_add")
 
 
-GLU_KINDS = {**ACTIVATIONS, "swigluoai": 3}
+GLU_KINDS = {"relu2": 0, "gelu_tanh": 1, "silu": 2, "swigluoai": 3}
 
 
 def glu_rows(gate_up: torch.Tensor, mid: torch.Tensor, kind: str, alpha: float = 1.702, limit: float = 7.0) -> None:
@@ -720,6 +786,54 @@ def retention_scan(qkv: torch.Tensor, decay: torch.Tensor, cos_sin: Optional[tor
              seg_slot.numel(), code(qkv.dtype), _stream()), "retention_scan")
 
 
+def token_shift(x: torch.Tensor, mu: torch.Tensor, out: torch.Tensor, state: torch.Tensor, token_seg: torch.Tensor,
+                seg_slot: torch.Tensor, seg_q_start: torch.Tensor) -> None:
+    """out[m, t, :] = x[t] + (x[t - 1] - x[t]) * mu[m] for every mix m (``mu`` ``[M, W]``, ``out`` ``[M, T, W]``).  The
+    input before a segment's first token is row ``slot`` of ``state`` (float32, its first W values), which
+    takes the segment's last input."""
+    _need(x, "x", contiguous=False)
+    _need(mu, "mu", torch.float32)
+    _need(out, "out", x.dtype)
+    _need(state, "state", torch.float32, contiguous=False)
+    for name, t in (("token_seg", token_seg), ("seg_slot", seg_slot), ("seg_q_start", seg_q_start)):
+        _need(t, name, torch.int32)
+    T, W = x.shape
+    M = mu.shape[0]
+    if mu.shape != (M, W) or out.shape != (M, T, W) or x.stride(1) != 1 or state.shape[1] < W or state.stride(1) != 1:
+        raise KernelError("token_shift: shapes do not match")
+    f = _fn("time_mixing", "ft_token_shift", "p q p p p q p p p i i i i")
+    _check(f(_ptr(x), x.stride(0), _ptr(mu), _ptr(out), _ptr(state), state.stride(0), _ptr(token_seg), _ptr(seg_slot),
+             _ptr(seg_q_start), T, W, M, code(x.dtype), _stream()), "token_shift")
+
+
+def time_mixing_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, w0: torch.Tensor,
+                     u: torch.Tensor, state: torch.Tensor, o: torch.Tensor, seg_slot: torch.Tensor,
+                     seg_q_start: torch.Tensor, heads: int, head_dim: int, key_dim: int) -> None:
+    """Per head, with ``w = exp(-exp(decay + w0))`` per key channel: ``o_t = (S + diag(u) k_t v_t^T)^T r_t``, then ``S
+    <- diag(w_t) S + k_t v_t^T``.  ``r`` and ``k`` are ``[T, heads * key_dim]``, ``v`` ``[T, heads * head_dim]`` (one
+    row stride), ``decay`` float32; the state of head h lies at ``h * head_dim * key_dim`` of its slot's row, ``[head_dim,
+    key_dim]``."""
+    for name, t in (("r", r), ("k", k), ("v", v)):
+        _need(t, name, r.dtype, contiguous=False)
+    for name, t in (("decay", decay), ("state", state)):
+        _need(t, name, torch.float32, contiguous=False)
+    for name, t in (("w0", w0), ("u", u), ("o", o)):
+        _need(t, name, torch.float32)
+    for name, t in (("seg_slot", seg_slot), ("seg_q_start", seg_q_start)):
+        _need(t, name, torch.int32)
+    T, kd, inner = r.shape[0], heads * key_dim, heads * head_dim
+    if r.shape != (T, kd) or k.shape != (T, kd) or v.shape != (T, inner) or decay.shape != (T, kd) \
+            or w0.numel() != kd or u.numel() != kd or o.shape != (T, inner) \
+            or state.shape[1] != inner * key_dim or state.stride(1) != 1:
+        raise KernelError("time_mixing_scan: shapes do not match")
+    if len({t.stride(0) for t in (r, k, v)}) != 1 or any(t.stride(1) != 1 for t in (r, k, v, decay)):
+        raise KernelError("time_mixing_scan: r, k and v need one row stride and unit column strides")
+    f = _fn("time_mixing", "ft_time_mixing_scan", "p p p q p q p p p q p p p i i i i i")
+    _check(f(_ptr(r), _ptr(k), _ptr(v), r.stride(0), _ptr(decay), decay.stride(0), _ptr(w0), _ptr(u), _ptr(state),
+             state.stride(0), _ptr(o), _ptr(seg_slot), _ptr(seg_q_start), heads, head_dim, key_dim,
+             seg_slot.numel(), code(r.dtype), _stream()), "time_mixing_scan")
+
+
 GATES = {"silu": 0, "sigmoid": 1}
 
 
@@ -792,6 +906,10 @@ def gemm_rows(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, *,
              float(act_limit), _stream()), "gemm_rows")
 
 
+# gated pairs the weight-streaming kernel applies to its accumulators
+GLU_ACTS = {"silu": 0, "swigluoai": 1, "gelu_tanh": 2}
+
+
 def skinny_gemm_takes(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor) -> bool:
     """Whether the weight-streaming tensor-core kernel takes these operands."""
     K = w.shape[-1]
@@ -807,10 +925,13 @@ def skinny_gemm(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, *,
                 c_rows: Optional[torch.Tensor] = None, row_scale: Optional[torch.Tensor] = None,
                 rows: Optional[int] = None, glu: bool = False, act: str = "silu",
                 act_alpha: float = 1.702, act_limit: float = 7.0, rows_per_pass: int = 8,
-                unary: Optional[str] = None) -> None:
+                unary: Optional[str] = None, bias: Optional[torch.Tensor] = None, group_rows: int = 0) -> None:
     """c = a @ w^T for few rows, streaming bfloat16 weights once through
     mma.sync; same conventions as :func:`gemm_rows`.  ``unary`` (one of
-    :data:`ACTIVATIONS`, without ``glu``): that function of the float32 accumulator is stored."""
+    :data:`ACTIVATIONS`, without ``glu``): that function of the float32 accumulator is stored; ``bias``
+    (float32 ``[N]``, without ``glu``) is added to the accumulator first.  ``group_rows``: ``w`` is ``[G, N, K]``
+    and rows ``g * group_rows ..`` of ``a`` and ``c`` belong to matrix g.  With ``glu``, ``act`` may be
+    ``silu``, ``swigluoai`` or ``gelu_tanh``."""
     _need(a, "a", torch.bfloat16, contiguous=False)
     _need(w, "w", torch.bfloat16)
     _need(c, "c", contiguous=False)
@@ -824,8 +945,16 @@ def skinny_gemm(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, *,
         raise KernelError("skinny_gemm: shapes do not match")
     if not skinny_gemm_takes(a, w, c):
         raise KernelError("skinny_gemm: needs bfloat16 operands, K % 8 == 0 and 16-byte aligned rows")
-    if (w.dim() == 3) != (group_offsets is not None):
-        raise KernelError("skinny_gemm: group_offsets must be given exactly for grouped ([G, N, K]) weights")
+    if (w.dim() == 3) != (group_offsets is not None or group_rows > 0):
+        raise KernelError("skinny_gemm: group_offsets or group_rows must be given exactly for grouped ([G, N, K]) weights")
+    if group_rows and (group_offsets is not None or M != G * group_rows or c.shape[0] < M):
+        raise KernelError("skinny_gemm: group_rows must divide the rows among the groups")
+    if bias is not None:
+        _need(bias, "bias", torch.float32)
+        if bias.numel() != N or glu:
+            raise KernelError("skinny_gemm: one bias per output, not with glu")
+    if act not in GLU_ACTS:
+        raise KernelError(f"skinny_gemm: activation {act!r} is not one of {sorted(GLU_ACTS)}")
     if rows_per_pass not in (8, 16, 32):
         raise KernelError("skinny_gemm: rows_per_pass must be 8, 16 or 32")
     if active is not None:
@@ -834,11 +963,12 @@ def skinny_gemm(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, *,
             raise KernelError("skinny_gemm: the active list needs G + 1 entries")
     if unary is not None and (glu or unary not in ACTIVATIONS):
         raise KernelError(f"skinny_gemm: cannot apply {unary!r} (with glu: {glu})")
-    f = _fn("skinny_gemm", "ft_skinny_gemm", "p q p q p i q p p p p p i i i i i i f f i i")
+    f = _fn("skinny_gemm", "ft_skinny_gemm", "p q p q p i q p p p p p i i i i i i f f i i p i")
     _check(f(_ptr(a), a.stride(0), _ptr(w), NW * K, _ptr(c), code(c.dtype), c.stride(0),
              _ptr(group_offsets), _ptr(active), _ptr(a_rows), _ptr(c_rows), _ptr(row_scale), M, N, K, G,
-             int(glu), 0 if act == "silu" else 1, float(act_alpha), float(act_limit),
-             rows_per_pass, 0 if unary is None else 1 + ACTIVATIONS[unary], _stream()), "skinny_gemm")
+             int(glu), GLU_ACTS[act], float(act_alpha), float(act_limit),
+             rows_per_pass, 0 if unary is None else 1 + ACTIVATIONS[unary], _ptr(bias), int(group_rows), _stream()),
+           "skinny_gemm")
 
 
 # ------------------------------------------------ grouped GEMM on tcgen05
@@ -1426,23 +1556,28 @@ def attn_prefill_mha(q: torch.Tensor, keys: torch.Tensor, shared_keys: Optional[
 # ---------------------------------------------------------------- router
 def router_select(logits: torch.Tensor, bias: Optional[torch.Tensor], ids: torch.Tensor,
                   weights: torch.Tensor, k: int, softmax_scoring: bool, renormalize: bool,
-                  scale: float, terms: int = 1, groups: int = 1, keep: int = 1) -> None:
+                  scale: float, terms: int = 1, groups: int = 1, keep: int = 1, group_top: int = 2,
+                  tail: Optional[torch.Tensor] = None) -> None:
     """Top-k of the scored router logits.  With ``terms`` > 1 a row of ``logits``
     holds that many partial logits per expert (``[T, terms * E]``), summed in
     order in float32 before scoring.  With ``groups`` > 1 the experts form that many equal
-    groups of neighbours, a group's value is the sum of its two largest choice values, and
-    only experts of the ``keep`` best groups can be chosen."""
+    groups of neighbours, a group's value is the sum of its ``group_top`` (2 or 1) largest choice values,
+    and only experts of the ``keep`` best groups can be chosen.  With ``tail`` (float32 ``[T]``) a row has
+    one more logit behind the experts' (per term), whose sigmoid goes there."""
     _need(logits, "logits", torch.float32)
     _need(ids, "ids", torch.int32)
     _need(weights, "weights", torch.float32)
     if bias is not None:
         _need(bias, "bias", torch.float32)
-    T, E = logits.shape[0], logits.shape[1] // terms
-    if logits.shape[1] != E * terms or not logits.is_contiguous():
+    T, E = logits.shape[0], logits.shape[1] // terms - (tail is not None)
+    if tail is not None:
+        _need(tail, "tail", torch.float32)
+    if logits.shape[1] % terms or E < 1 or not logits.is_contiguous() or (tail is not None and tail.numel() < T):
         raise KernelError(f"router_select: logits {tuple(logits.shape)} do not hold {terms} terms per expert")
-    f = _fn("moe_route", "ft_router_select", "p p p p i i i i i f i i i")
+    f = _fn("moe_route", "ft_router_select", "p p p p i i i i i f i i i i p")
     _check(f(_ptr(logits), _ptr(bias), _ptr(ids), _ptr(weights), T, E, k, int(softmax_scoring),
-             int(renormalize), float(scale), int(terms), int(groups), int(keep), _stream()), "router_select")
+             int(renormalize), float(scale), int(terms), int(groups), int(keep), int(group_top), _ptr(tail), _stream()),
+           "router_select")
 
 
 ROUTE_SMALL_MAX_T = 8
@@ -1457,7 +1592,7 @@ def route_small(logits: torch.Tensor, bias: Optional[torch.Tensor], ids: torch.T
                 weights: torch.Tensor, counts: torch.Tensor, offsets: torch.Tensor,
                 sorted_route: torch.Tensor, sorted_token: torch.Tensor, active: torch.Tensor, k: int,
                 softmax_scoring: bool, renormalize: bool, scale: float, terms: int = 1, groups: int = 1,
-                keep: int = 1, busy_of: int = 0) -> None:
+                keep: int = 1, busy_of: int = 0, group_top: int = 2, tail: Optional[torch.Tensor] = None) -> None:
     """:func:`router_select` and :func:`moe_sort` in one launch (same results)."""
     _need(logits, "logits", torch.float32)
     _need(weights, "weights", torch.float32)
@@ -1466,18 +1601,22 @@ def route_small(logits: torch.Tensor, bias: Optional[torch.Tensor], ids: torch.T
     for name, t in (("ids", ids), ("counts", counts), ("offsets", offsets),
                     ("sorted_route", sorted_route), ("sorted_token", sorted_token), ("active", active)):
         _need(t, name, torch.int32)
-    T, E = logits.shape[0], logits.shape[1] // terms
+    T, E = logits.shape[0], logits.shape[1] // terms - (tail is not None)
+    if tail is not None:
+        _need(tail, "tail", torch.float32)
     R = T * k
     busy_of = busy_of or E
-    if logits.shape[1] != E * terms or not route_small_takes(T, E, k) or not 1 <= busy_of <= E:
+    if logits.shape[1] % terms or E < 1 or (tail is not None and tail.numel() < T) \
+            or not route_small_takes(T, E, k) or not 1 <= busy_of <= E:
         raise KernelError(f"route_small: refuses {T} tokens, {E} experts, top-{k}")
     if counts.numel() < E or offsets.numel() < E + 1 or sorted_route.numel() < R \
             or sorted_token.numel() < R or active.numel() < busy_of + 1 or ids.numel() < R or weights.numel() < R:
         raise KernelError("route_small: output buffers are too small")
-    f = _fn("moe_route", "ft_route_small", "p p p p p p p p p i i i i i i f i i i")
+    f = _fn("moe_route", "ft_route_small", "p p p p p p p p p i i i i i i f i i i i p")
     _check(f(_ptr(logits), _ptr(bias), _ptr(ids), _ptr(weights), _ptr(counts), _ptr(offsets),
              _ptr(sorted_route), _ptr(sorted_token), _ptr(active), T, E, busy_of, k, int(softmax_scoring),
-             int(renormalize), float(scale), int(terms), int(groups), int(keep), _stream()), "route_small")
+             int(renormalize), float(scale), int(terms), int(groups), int(keep), int(group_top),
+             _ptr(tail), _stream()), "route_small")
 
 
 def router_logits_takes(x: torch.Tensor, w: torch.Tensor) -> bool:

@@ -234,6 +234,7 @@ __device__ __forceinline__ float act_apply(float x, int kind) {
   switch (kind) {
     case 0: { const float r = fmaxf(x, 0.f); return r * r; }                     // relu squared
     case 1: return 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));  // tanh-GELU
+    case 4: return tanhf(x);                                                       // (3: a pair, see glu_rows)
     default: return x / (1.f + expf(-x));                                         // SiLU
   }
 }
@@ -270,8 +271,11 @@ __global__ void __launch_bounds__(256) softcap_kernel(float* __restrict__ x, lon
 // ------------------------------------------------- what a feed-forward hands on, row by row
 // A branch output of a token is a sum of rows that nobody has added yet (float32, in this order):
 //   z = sum_j s_j * rows[t, j, :]      the k partial rows (s_j = 1 without scales)
-//     + extra[t, :]                     one more row per token (a shared expert), if there is one
+//     + g_t * extra[t, :]               one more row per token (a shared expert), if there is one (g_t = 1
+//                                       without a gate per token)
 //     + c_t * source[t, :]              c_t = sum of weights[t, j] over the slots whose id is >= experts
+//     + sum_j b_j * beside[t, j, :]     rows of another sublayer that reads the same input (b_j = 1 without
+//                                       scales), if there is one
 // With ids, slots whose id is >= `experts` have no row (it is never written, so it is not read): such
 // a slot hands the branch's own input back, times its weight.
 struct BranchArgs {
@@ -281,7 +285,10 @@ struct BranchArgs {
   const float* weights;    // [T, k]
   const void* source;      // [T, H]
   const void* extra;       // [T, H] or nullptr
-  int k, experts;
+  const float* extra_gate; // [T] or nullptr
+  const void* beside;      // [T, kb, H] or nullptr
+  const float* beside_scale;  // [kb] or nullptr
+  int k, experts, kb;
 };
 
 __device__ __forceinline__ void store4f(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
@@ -305,8 +312,14 @@ __device__ __forceinline__ float branch_at(const BranchArgs& b, int t, int H, in
     const float v = to_float(rows[(size_t)j * H]);
     z = b.part_scale ? fmaf(b.part_scale[j], v, z) : z + v;
   }
-  if (b.extra) z += to_float(((const AT*)b.extra)[(size_t)t * H + c]);
+  if (b.extra) z = fmaf(b.extra_gate ? b.extra_gate[t] : 1.f, to_float(((const AT*)b.extra)[(size_t)t * H + c]), z);
   if (back != 0.f) z = fmaf(back, to_float(((const AT*)b.source)[(size_t)t * H + c]), z);
+  if (b.beside) {
+    const AT* other = (const AT*)b.beside + (size_t)t * b.kb * H + c;
+    float y = 0.f;
+    for (int j = 0; j < b.kb; ++j) y = fmaf(b.beside_scale ? b.beside_scale[j] : 1.f, to_float(other[(size_t)j * H]), y);
+    z += y;
+  }
   return z;
 }
 // Which slots of token t have a row (bit j), and c_t; every lane of the (whole) warp gets both.  The ids are
@@ -325,8 +338,20 @@ template <typename AT>
 __device__ __forceinline__ float4 branch_at4(const BranchArgs& b, int t, int H, int gi, unsigned slots, float back) {
   const AT* rows = (const AT*)b.rows + (size_t)t * b.k * H + 4 * gi;
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-  float4 z = zero, e = zero, h = zero;
-  if (b.extra) e = load4f((const AT*)b.extra + (size_t)t * H + 4 * gi);
+  float4 z = zero, e = zero, h = zero, y = zero;
+  float eg = 1.f;
+  if (b.extra) {
+    e = load4f((const AT*)b.extra + (size_t)t * H + 4 * gi);
+    if (b.extra_gate) eg = b.extra_gate[t];
+  }
+  if (b.beside) {
+    const AT* other = (const AT*)b.beside + (size_t)t * b.kb * H + 4 * gi;
+    for (int j = 0; j < b.kb; ++j) {
+      const float4 v = load4f(other + (size_t)j * H);
+      const float s = b.beside_scale ? b.beside_scale[j] : 1.f;
+      y.x = fmaf(s, v.x, y.x); y.y = fmaf(s, v.y, y.y); y.z = fmaf(s, v.z, y.z); y.w = fmaf(s, v.w, y.w);
+    }
+  }
   if (back != 0.f) h = load4f((const AT*)b.source + (size_t)t * H + 4 * gi);
   for (int j0 = 0; j0 < b.k; j0 += 4) {
     float4 v[4];
@@ -338,8 +363,9 @@ __device__ __forceinline__ float4 branch_at4(const BranchArgs& b, int t, int H, 
       z.x = fmaf(s, v[u].x, z.x); z.y = fmaf(s, v[u].y, z.y); z.z = fmaf(s, v[u].z, z.z); z.w = fmaf(s, v[u].w, z.w);
     }
   }
-  z.x += e.x; z.y += e.y; z.z += e.z; z.w += e.w;
+  z.x = fmaf(eg, e.x, z.x); z.y = fmaf(eg, e.y, z.y); z.z = fmaf(eg, e.z, z.z); z.w = fmaf(eg, e.w, z.w);
   z.x = fmaf(back, h.x, z.x); z.y = fmaf(back, h.y, z.y); z.z = fmaf(back, h.z, z.z); z.w = fmaf(back, h.w, z.w);
+  z.x += y.x; z.y += y.y; z.z += y.z; z.w += y.w;
   return z;
 }
 
@@ -496,6 +522,107 @@ __global__ void __launch_bounds__(256) norm_add_kernel(NormAddArgs a) {
     const float inv2 = 1.0f / sqrtf(ss2 / (float)H + a.next_eps);
     for (int i = threadIdx.x; i < H; i += blockDim.x)
       o[i] = from_float<AT>(row[i] * inv2 * (a.next_weight[i] + one2));
+  }
+}
+
+// ------------------------------------- a branch joins the residual, then layer norms of the sum
+// x[t, :] += z of token t (without a branch: x stays); then, with the mean and the variance (the mean of the
+// squared deviations) of the new row taken once,
+//   out1 = (x - mean) / sqrt(var + eps1) * w1 [+ b1]     and, with a second weight,
+//   out2 = (x - mean) / sqrt(var + eps2) * w2 [+ b2]
+// for two sublayers that read the same row through norms of their own.  One block per token; the row stays
+// in registers between the passes (KEEP > 0: 4 * blockDim * KEEP values, every row 16-byte aligned, all loads
+// in flight together), or in shared memory (KEEP = 0: any row).
+struct JoinNormArgs {
+  BranchArgs b;            // b.rows nullptr: no branch
+  float* residual;
+  const float *w1, *b1, *w2, *b2;
+  void *out1, *out2;
+  int H;
+  float eps1, eps2;
+};
+
+template <typename AT, int KEEP, int THREADS>
+__global__ void __launch_bounds__(THREADS) join_layer_norm_kernel(JoinNormArgs a) {
+  extern __shared__ float row[];
+  __shared__ float scratch[33];
+  pdl_wait();
+  const int t = blockIdx.x, H = a.H;
+  float* r = a.residual + (size_t)t * H;
+  AT* o1 = (AT*)a.out1 + (size_t)t * H;
+  AT* o2 = (AT*)a.out2 + (size_t)t * H;
+  const bool two = a.w2 != nullptr;
+  float sum = 0.f, sq = 0.f;
+  if constexpr (KEEP > 0) {
+    float4 x[KEEP];
+    const int groups = H >> 2;
+    float back = 0.f;
+    const unsigned slots = a.b.rows ? branch_slots(a.b, t, back) : 0u;
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+      const int gi = threadIdx.x + j * THREADS;
+      x[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (gi < groups) {
+        x[j] = load4f(r + 4 * gi);
+        if (a.b.rows) {
+          const float4 z = branch_at4<AT>(a.b, t, H, gi, slots, back);
+          x[j].x += z.x; x[j].y += z.y; x[j].z += z.z; x[j].w += z.w;
+          store4f(r + 4 * gi, x[j]);
+        }
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) sum += (x[j].x + x[j].y) + (x[j].z + x[j].w);
+    const float mean = block_sum(sum, scratch) / (float)H;
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+      if ((int)threadIdx.x + j * THREADS < groups) {
+        x[j].x -= mean; x[j].y -= mean; x[j].z -= mean; x[j].w -= mean;
+        sq = fmaf(x[j].x, x[j].x, sq); sq = fmaf(x[j].y, x[j].y, sq);
+        sq = fmaf(x[j].z, x[j].z, sq); sq = fmaf(x[j].w, x[j].w, sq);
+      }
+    }
+    const float var = block_sum(sq, scratch) / (float)H;
+    auto write = [&](AT* o, const float* w, const float* b, float eps) {
+      const float inv = 1.f / sqrtf(var + eps);
+#pragma unroll
+      for (int j = 0; j < KEEP; ++j) {
+        const int gi = threadIdx.x + j * THREADS;
+        if (gi < groups) {
+          const float4 wv = load4f(w + 4 * gi);
+          float4 v = make_float4(x[j].x * inv * wv.x, x[j].y * inv * wv.y, x[j].z * inv * wv.z, x[j].w * inv * wv.w);
+          if (b) {
+            const float4 bv = load4f(b + 4 * gi);
+            v.x += bv.x; v.y += bv.y; v.z += bv.z; v.w += bv.w;
+          }
+          store4f(o + 4 * gi, v);
+        }
+      }
+    };
+    write(o1, a.w1, a.b1, a.eps1);
+    if (two) write(o2, a.w2, a.b2, a.eps2);
+  } else {
+    for (int i = threadIdx.x; i < H; i += THREADS) {
+      float v = r[i];
+      if (a.b.rows) {
+        v += branch_at<AT>(a.b, t, H, i);
+        r[i] = v;
+      }
+      row[i] = v;
+      sum += v;
+    }
+    const float mean = block_sum(sum, scratch) / (float)H;
+    for (int i = threadIdx.x; i < H; i += THREADS) {
+      const float d = row[i] - mean;
+      row[i] = d;
+      sq = fmaf(d, d, sq);
+    }
+    const float var = block_sum(sq, scratch) / (float)H;
+    const float inv1 = 1.f / sqrtf(var + a.eps1), inv2 = 1.f / sqrtf(var + a.eps2);
+    for (int i = threadIdx.x; i < H; i += THREADS) {
+      o1[i] = from_float<AT>(row[i] * inv1 * a.w1[i] + (a.b1 ? a.b1[i] : 0.f));
+      if (two) o2[i] = from_float<AT>(row[i] * inv2 * a.w2[i] + (a.b2 ? a.b2[i] : 0.f));
+    }
   }
 }
 
@@ -1024,7 +1151,7 @@ int ft_gate_heads(void* o, const void* z, long long ldz, int heads, int d, int d
 
 int ft_activation(void* x, long long n, int kind, int dtype, cudaStream_t stream) {
   if (n <= 0) return FT_OK;
-  if (kind < 0 || kind > 2) return FT_ERR_SHAPE;
+  if (kind < 0 || kind > 4 || kind == 3) return FT_ERR_SHAPE;
   if (dtype == FT_DTYPE_BF16 && !(n & 7) && !((uintptr_t)x & 15)) {
     const long long n8 = n >> 3;
     launch_pdl(activation_bf16x8_kernel, dim3((unsigned)((n8 + 255) / 256)), dim3(256), 0, stream, (uint4*)x, n8,
@@ -1047,30 +1174,32 @@ int ft_softcap(float* x, long long n, float cap, cudaStream_t stream) {
   return FT_OK;
 }
 
-static int branch_args(BranchArgs& b, const void* rows, int k, const float* part_scale, const int* ids,
-                       const float* weights, int experts, const void* source, const void* extra) {
-  if (!rows || k <= 0 || (ids && (!weights || !source || part_scale || experts < 0))) return FT_ERR_SHAPE;
-  b = BranchArgs{rows, part_scale, ids, weights, source, extra, k, experts};
+// `b` comes from the caller as a whole (host memory, read during the call)
+static int branch_check(const BranchArgs* b) {
+  if (!b || !b->rows || b->k <= 0 || (b->ids && (!b->weights || !b->source || b->part_scale || b->experts < 0)))
+    return FT_ERR_SHAPE;
+  if ((b->extra_gate && !b->extra) || (b->beside && b->kb <= 0) || (b->beside_scale && !b->beside)) return FT_ERR_SHAPE;
   return FT_OK;
 }
+static bool branch_aligned(const BranchArgs& b) {
+  return !((uintptr_t)b.rows & 15) && !((uintptr_t)b.source & 15) && !((uintptr_t)b.extra & 15) && !((uintptr_t)b.beside & 15);
+}
 
-int ft_norm_add(const void* branch, int k, const float* part_scale, const int* ids, const float* route_weights,
-                int experts, const void* source, const void* extra, const float* weight, int plus_one, float eps,
-                float mult, float* residual, const float* next_weight, int next_plus_one, float next_eps,
+int ft_norm_add(const BranchArgs* branch, const float* weight, int plus_one, float eps, float mult, float* residual, const float* next_weight, int next_plus_one, float next_eps,
                 void* next_out, void* copy_out, long long copy_ld, int T, int H, int dtype, cudaStream_t stream) {
   if (T <= 0) return FT_OK;
   NormAddArgs a{};
-  const int rc = branch_args(a.b, branch, k, part_scale, ids, route_weights, experts, source, extra);
+  const int rc = branch_check(branch);
   if (rc != FT_OK) return rc;
+  a.b = *branch;
   if (H <= 0 || H > 12288) return FT_ERR_SHAPE;
   a.weight = weight; a.residual = residual; a.next_weight = next_weight; a.next_out = next_out;
   a.copy_out = copy_out; a.copy_ld = copy_ld; a.plus_one = plus_one; a.next_plus_one = next_plus_one; a.H = H;
   a.eps = eps; a.next_eps = next_eps; a.mult = mult;
-  const bool vec = !(H & 3) && H <= 4 * 256 * NORM_ADD_KEEP && !((uintptr_t)branch & 15) && !((uintptr_t)weight & 15) &&
+  const bool vec = !(H & 3) && H <= 4 * 256 * NORM_ADD_KEEP && branch_aligned(a.b) && !((uintptr_t)weight & 15) &&
                    !((uintptr_t)residual & 15) && !((uintptr_t)next_weight & 15) && !((uintptr_t)next_out & 15) &&
-                   !((uintptr_t)source & 15) && !((uintptr_t)extra & 15) && !((uintptr_t)copy_out & 15) &&
-                   !(copy_ld & 3);
-  if (vec && k <= 32) {
+                   !((uintptr_t)copy_out & 15) && !(copy_ld & 3);
+  if (vec && a.b.k <= 32) {
     const dim3 g(T), th(256);
     if (H <= 1024) { FT_DISPATCH(dtype, AT, (launch_pdl(norm_add_kernel<AT, 1>, g, th, 0, stream, a))); }
     else if (H <= 2048) { FT_DISPATCH(dtype, AT, (launch_pdl(norm_add_kernel<AT, 2>, g, th, 0, stream, a))); }
@@ -1084,12 +1213,40 @@ int ft_norm_add(const void* branch, int k, const float* part_scale, const int* i
   return FT_OK;
 }
 
-int ft_branch_sum(const void* branch, int k, const int* ids, const float* route_weights, int experts,
-                  const void* source, const void* extra, void* out, int T, int H, int dtype, cudaStream_t stream) {
+// branch nullptr: only the norms; w2 nullptr: one norm
+int ft_join_layer_norm(const BranchArgs* branch, float* residual, const float* w1, const float* b1, float eps1,
+                       void* out1, const float* w2, const float* b2, float eps2, void* out2, int T, int H, int dtype,
+                       cudaStream_t stream) {
   if (T <= 0) return FT_OK;
-  BranchArgs b;
-  const int rc = branch_args(b, branch, k, nullptr, ids, route_weights, experts, source, extra);
+  JoinNormArgs a{};
+  if (branch) {
+    const int rc = branch_check(branch);
+    if (rc != FT_OK) return rc;
+    a.b = *branch;
+  }
+  if (H <= 0 || H > 12288 || !residual || !w1 || !out1 || (w2 && !out2)) return FT_ERR_SHAPE;
+  a.residual = residual; a.w1 = w1; a.b1 = b1; a.w2 = w2; a.b2 = b2; a.out1 = out1; a.out2 = out2; a.H = H;
+  a.eps1 = eps1; a.eps2 = eps2;
+  const bool vec = !(H & 3) && H <= 8192 && branch_aligned(a.b) && a.b.k <= 32 && !((uintptr_t)residual & 15) &&
+                   !((uintptr_t)w1 & 15) && !((uintptr_t)b1 & 15) && !((uintptr_t)w2 & 15) && !((uintptr_t)b2 & 15) &&
+                   !((uintptr_t)out1 & 15) && !((uintptr_t)out2 & 15);
+  const dim3 g(T), th(256);
+  if (vec && H <= 1024) { FT_DISPATCH(dtype, AT, (launch_pdl(join_layer_norm_kernel<AT, 1, 256>, g, th, 0, stream, a))); }
+  else if (vec && H <= 2048) { FT_DISPATCH(dtype, AT, (launch_pdl(join_layer_norm_kernel<AT, 2, 256>, g, th, 0, stream, a))); }
+  else if (vec && H <= 4096) { FT_DISPATCH(dtype, AT, (launch_pdl(join_layer_norm_kernel<AT, 4, 256>, g, th, 0, stream, a))); }
+  else if (vec) { FT_DISPATCH(dtype, AT, (launch_pdl(join_layer_norm_kernel<AT, 8, 256>, g, th, 0, stream, a))); }
+  else {
+    FT_DISPATCH(dtype, AT, (launch_pdl(join_layer_norm_kernel<AT, 0, 256>, g, th, (size_t)H * sizeof(float), stream, a)));
+  }
+  FT_LAUNCH_CHECK();
+  return FT_OK;
+}
+
+int ft_branch_sum(const BranchArgs* branch, void* out, int T, int H, int dtype, cudaStream_t stream) {
+  if (T <= 0) return FT_OK;
+  const int rc = branch_check(branch);
   if (rc != FT_OK) return rc;
+  const BranchArgs b = *branch;
   const long long n = (long long)T * H;
   FT_DISPATCH(dtype, AT,
               (launch_pdl(branch_sum_kernel<AT>, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, b,
@@ -1098,19 +1255,19 @@ int ft_branch_sum(const void* branch, int k, const int* ids, const float* route_
   return FT_OK;
 }
 
-int ft_cast_rows(float* x, const void* branch, int k, const int* ids, const float* route_weights, int experts,
-                 const void* source, const void* extra, void* dst, long long ld, int T, int H, int dtype,
+int ft_cast_rows(float* x, const BranchArgs* branch, void* dst, long long ld, int T, int H, int dtype,
                  cudaStream_t stream) {
   if (T <= 0 || H <= 0) return FT_OK;
   BranchArgs b{};
   if (branch) {
-    const int rc = branch_args(b, branch, k, nullptr, ids, route_weights, experts, source, extra);
+    const int rc = branch_check(branch);
     if (rc != FT_OK) return rc;
+    b = *branch;
   }
   const long long n = (long long)T * H;
   const int groups = H / 4;
-  if (!(H & 3) && !(ld & 3) && !((uintptr_t)x & 15) && !((uintptr_t)dst & 15) && !((uintptr_t)branch & 15) &&
-      !((uintptr_t)source & 15) && !((uintptr_t)extra & 15) && k <= 32) {
+  if (!(H & 3) && !(ld & 3) && !((uintptr_t)x & 15) && !((uintptr_t)dst & 15) && branch_aligned(b) &&
+      b.k <= 32) {
     FT_DISPATCH(dtype, AT,
                 (launch_pdl(cast_rows4_kernel<AT>, dim3(T), dim3(256), 0, stream, x, b, (AT*)dst, ld, groups)));
   } else {

@@ -15,7 +15,8 @@
 // not depend on the launch shape.  Grouped use (experts): blockIdx.y is the
 // j-th expert that has tokens (from the `active` list, so the grid is no larger
 // than the number of routes), rows group_offsets[e]..group_offsets[e+1] of the
-// sorted routes are its tokens, taken 8*NT at a time.
+// sorted routes are its tokens, taken 8*NT at a time.  Without those lists `group_rows` rows of A follow
+// one another for every group: several matrices of one shape, each against rows of its own, in one launch.
 //
 // Reference counterpart: python/freetoken/kernel/triton/decode_moe.py:5-75 (one
 // program per route, CUDA-core FMAs: an expert's weights are read once per
@@ -38,7 +39,9 @@ struct SkinnyArgs {
   int M, N, K, G;
   int act;
   float act_alpha, act_limit;
-  int unary = 0;             // without GLU: 0 nothing, 1 relu(x)^2, 2 tanh-GELU, 3 SiLU on the accumulator
+  int unary = 0;             // without GLU: 0 nothing, 1 relu(x)^2, 2 tanh-GELU, 3 SiLU, 5 tanh on the accumulator
+  const float* bias = nullptr;   // [N], added to the accumulator (not with GLU)
+  int group_rows = 0;            // > 0: every group has that many rows, group g the rows g * group_rows ..
 };
 
 __device__ __forceinline__ uint4 ld_stream(const uint4* p) {
@@ -60,6 +63,7 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], unsigned a0, unsigned a1
 
 __device__ __forceinline__ float glu_act_s(float g, float u, int act, float alpha, float limit) {
   if (act == 0) return (g / (1.f + __expf(-g))) * u;
+  if (act == 2) return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
   return (g / (1.f + __expf(-alpha * g))) * (u + 1.f);
@@ -70,6 +74,7 @@ __device__ __forceinline__ float unary_act_s(float x, int kind) {
     case 1: { const float r = fmaxf(x, 0.f); return r * r; }
     case 2: return 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
     case 3: return x / (1.f + expf(-x));
+    case 5: return tanhf(x);
     default: return x;
   }
 }
@@ -95,6 +100,10 @@ __global__ void __launch_bounds__(KS * 32) skinny_kernel(SkinnyArgs a) {
     group = a.active[blockIdx.y];
   }
   int row_begin = 0, row_end = a.M;
+  if (a.group_rows) {
+    row_begin = group * a.group_rows;
+    row_end = row_begin + a.group_rows;
+  }
   if (a.group_offsets) {
     row_begin = a.group_offsets[group];
     row_end = a.group_offsets[group + 1];
@@ -190,6 +199,7 @@ __global__ void __launch_bounds__(KS * 32) skinny_kernel(SkinnyArgs a) {
       const int row = pass + 8 * j + tok, n = n0 + r;
       if (row < row_end && n < a.N) {
         const int crow = a.c_rows ? a.c_rows[row] : row;
+        if (!GLU && a.bias) s += a.bias[n];
         float v = GLU ? glu_act_s(s, su, a.act, a.act_alpha, a.act_limit) : (a.unary ? unary_act_s(s, a.unary) : s);
         if (a.row_scale) v *= a.row_scale[crow];
         C[(size_t)crow * a.ldc + n] = from_float<OT>(v);
@@ -238,25 +248,31 @@ extern "C" int ft_skinny_gemm(const void* A, long long lda, const void* W,
                               const int* group_offsets, const int* active, const int* a_rows,
                               const int* c_rows, const float* row_scale, int M, int N, int K, int G, int glu,
                               int act, float act_alpha, float act_limit, int rows_per_pass, int unary,
-                              cudaStream_t stream) {
+                              const float* bias, int group_rows, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return FT_OK;
   if (K <= 0 || (K & 7) || (lda & 7) || G <= 0) return FT_ERR_SHAPE;
   if (((uintptr_t)A & 15) || ((uintptr_t)W & 15) || ((w_group_stride * 2) & 15)) return FT_ERR_SHAPE;
   if (G > 65535) return FT_ERR_SHAPE;
   SkinnyArgs a{(const __nv_bfloat16*)A, (const __nv_bfloat16*)W, C, group_offsets, active, a_rows,
                c_rows, row_scale, lda, ldc, w_group_stride, M, N, K, G, act, act_alpha, act_limit};
-  if (unary < 0 || unary > 3 || (glu && unary)) return FT_ERR_SHAPE;
+  if (unary < 0 || unary > 5 || unary == 4 || (glu && unary) || (glu && bias) || act < 0 || act > 2) return FT_ERR_SHAPE;
+  if (group_rows < 0 || (group_rows && (group_offsets || active || (long long)group_rows * G > M))) return FT_ERR_SHAPE;
   a.unary = unary;
+  a.bias = bias;
+  a.group_rows = group_rows;
   // with the list of busy groups, no more groups than rows can have any
   dim3 grid((N + 15) / 16, active ? min(G, M) : G);
   const int nt = rows_per_pass / 8;
   int rc;
-  int ks = (!glu && !group_offsets && G == 1) ? dense_k_split(N, K) : 4;
+  int ks = (!group_offsets && (G == 1 || group_rows)) ? dense_k_split(N * G * (glu ? 2 : 1), K) : 4;
   // an expert's down projection has short rows: two warps a block keep a warp's stream
   // of a row long enough (a function of the weight's shape, like the dense choice)
   if (!glu && group_offsets && K <= 2048) ks = 2;
   if (c_dtype == FT_DTYPE_BF16) {
-    if (glu) rc = launch_nt<true, __nv_bfloat16, 2>(a, nt, grid, stream);
+    // gate and up rows side by side: the experts' blocks take 2 warps, a dense layer's as many as split its rows
+    if (glu && !group_offsets && ks >= 8) rc = launch_nt<true, __nv_bfloat16, 8>(a, nt, grid, stream);
+    else if (glu && !group_offsets && ks == 4) rc = launch_nt<true, __nv_bfloat16, 4>(a, nt, grid, stream);
+    else if (glu) rc = launch_nt<true, __nv_bfloat16, 2>(a, nt, grid, stream);
     else if (ks == 2) rc = launch_nt<false, __nv_bfloat16, 2>(a, nt, grid, stream);
     else if (ks == 16) rc = launch_nt<false, __nv_bfloat16, 16>(a, nt, grid, stream);
     else if (ks == 8) rc = launch_nt<false, __nv_bfloat16, 8>(a, nt, grid, stream);

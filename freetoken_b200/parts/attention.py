@@ -9,7 +9,7 @@ them, or the latest ``sliding_window``), then ``@ Wo^T``.
 Options no model of the reference has, each a parameter of the mixer: a short causal
 convolution per channel behind the q, k and v projections (its last inputs per request in a
 state slot); a mask in chunks (a query sees the keys of its own chunk of positions); scores
-capped by ``cap * tanh(s / cap)``; a sink in the softmax's denominator, a fixed score or a
+capped by ``cap * tanh(s / cap)``; values blended with an earlier layer's; a sink in the softmax's denominator, a fixed score or a
 learned one per head; a sigmoid gate on the heads' outputs, one per head or one per value, read
 from the mixer's input by the same merged product.
 
@@ -140,7 +140,7 @@ class PagedAttention(PagedSoftmaxCore, Mixer):
     the weights are bound, which changes no score and no output and costs cache and
     arithmetic only where the two sizes differ.  ``bias`` (default False): the q, k, v and o
     projections add a bias (``checkpoint_names`` then also has q_bias, k_bias, v_bias, o_bias
-    and the fused qkv_bias).
+    and the fused qkv_bias); ``o_bias`` (default: as ``bias``): whether the o projection does.
 
     ``conv_taps`` (default 0): q, k and v each pass a causal convolution over time per channel
     (``checkpoint_names`` q_conv, k_conv, v_conv: ``[channels, taps]``, the last column weighing
@@ -151,6 +151,10 @@ class PagedAttention(PagedSoftmaxCore, Mixer):
     head, ``checkpoint_names`` sink): a score without key or value in the softmax's denominator.
     ``gate`` (``"head"`` or ``"element"``): the heads' outputs times ``sigmoid(Wg x)``, one gate
     per head or per value (``checkpoint_names`` gate), merged into the qkv product.
+    ``value_mix`` (None, ``"source"`` or ``"blend"``): in every layer that says ``"blend"`` the values become ``(1 -
+    lambda) v + lambda v_s`` before they are cached, ``v_s`` the values of the same token in the layer that says
+    ``"source"`` (it runs earlier in the schedule and has as many KV heads and as large values) and ``lambda`` a
+    learned number (``checkpoint_names`` value_mix, shape ``[]``; the source's own, where it exists, is unused).
     ``fill_heads`` (default False): in bfloat16, heads of up to 128 values that are no size of the
     tensor-core attention kernels (32, 64, 128) are filled up with zeros to the next one, exactly as
     heads are filled up to the larger of key and value size: a model with heads of 112 values then
@@ -211,11 +215,18 @@ class PagedAttention(PagedSoftmaxCore, Mixer):
         self._split_conv = [f"{self.scope}.{names[k]}" for k in ("q_conv", "k_conv", "v_conv")] if self.taps else []
         self.w_conv = self.w_sink = None
         self.gate_width = 0 if not self.gate else (self.nq if self.gate == "head" else self.nq * self.dv)
-        if self.gate and self.has_bias:
-            raise ValueError("a gate merged into a biased qkv product is not offered")
+        self.has_o_bias = bool(p.get("o_bias", self.has_bias))
+        self.value_mix = p.get("value_mix")
+        if self.value_mix not in (None, "source", "blend"):
+            raise ValueError("value_mix must be None, 'source' or 'blend'")
+        if self.value_mix and self.taps:
+            raise ValueError("values blended across layers beside a convolution are not offered")
+        self.n_value_mix = f"{self.scope}.{names['value_mix']}" if self.value_mix else None
+        self.w_value_mix = None
+        if self.has_o_bias:
+            self.n_o_bias = f"{self.scope}.{names['o_bias']}"
         if self.has_bias:
             self.n_qkv_bias = f"{self.scope}.{names['qkv_bias']}"
-            self.n_o_bias = f"{self.scope}.{names['o_bias']}"
             self._split_bias = [f"{self.scope}.{names[k]}" for k in ("q_bias", "k_bias", "v_bias")]
 
     def children(self):
@@ -252,6 +263,10 @@ class PagedAttention(PagedSoftmaxCore, Mixer):
             specs.append(TensorSpec(self.n_qkv_bias, (qn + kn + vn,), role="small32", tag="bias", sources=(Cat((
                 Name(self._split_bias[0], (qn,)), Name(self._split_bias[1], (kn,)),
                 Name(self._split_bias[2], (vn,))), 0),)))
+        if self.value_mix:
+            specs.append(TensorSpec(self.n_value_mix, (), role="small32", init=Init(0.4, 0.1), tag="value_mix",
+                                    optional=self.value_mix == "source", keep=self.value_mix == "blend"))
+        if self.has_o_bias:
             specs.append(TensorSpec(self.n_o_bias, (self.hidden,), role="small32", tag="bias"))
         if self.norm_mode:
             sizes = (qn, kn) if self.norm_mode == 1 else (self.dk, self.dk)
@@ -298,7 +313,12 @@ class PagedAttention(PagedSoftmaxCore, Mixer):
         self.w_o = self._filled(tensors[self.n_o], ((self.nq, self.dv),), 1)
         if self.has_bias:
             self.b_qkv = self._filled(tensors[self.n_qkv_bias], runs, 0)
+            if self.gate:              # the gate's rows of the merged product have no bias
+                self.b_qkv = torch.cat((self.b_qkv, self.b_qkv.new_zeros(self.w_qkv.shape[0] - self.b_qkv.numel())))
+        if self.has_o_bias:
             self.b_o = tensors[self.n_o_bias]
+        if self.value_mix == "blend":
+            self.w_value_mix = tensors[self.n_value_mix]
         if self.norm_mode == 1:
             self.w_qnorm = self._filled(tensors[self.n_qnorm], ((self.nq, self.dk),), 0)
             self.w_knorm = self._filled(tensors[self.n_knorm], ((self.nkv, self.dk),), 0)
@@ -313,7 +333,7 @@ class PagedAttention(PagedSoftmaxCore, Mixer):
             self.options = ops.ScoreOptions(self.chunk, self.softcap, self.sink_value, self.w_sink)
 
     def libraries(self, dtype) -> List[str]:
-        return (["elementwise"] + self.attention_libraries(dtype, self._head_size(dtype)) + linear.libraries(dtype, self.has_bias)
+        return (["elementwise"] + self.attention_libraries(dtype, self._head_size(dtype)) + linear.libraries(dtype, self.has_bias or self.has_o_bias)
                 + (["recurrent"] if self.taps else []) + (["rowwise"] if self.gate else []))
 
     # ---- forward ----------------------------------------------------------------
@@ -322,7 +342,9 @@ class PagedAttention(PagedSoftmaxCore, Mixer):
         ws = ctx.workspace
         qn, kn = self.nq * self.d, self.nkv * self.d
         gw = self.gate_width if self.gate == "head" else (qn if self.gate else 0)
-        qkv = linear.linear(x, self.w_qkv, ws.get("attn.qkv", (T, qn + 2 * kn + gw), ctx.dtype), bias=self.b_qkv)
+        # the rows of a layer whose values later layers blend in stay until the step is over
+        rows = "attn.qkv_source" if self.value_mix == "source" else "attn.qkv"
+        qkv = linear.linear(x, self.w_qkv, ws.get(rows, (T, qn + 2 * kn + gw), ctx.dtype), bias=self.b_qkv)
         gate = qkv[:, qn + 2 * kn:] if self.gate else None
         if self.gate:
             qkv = qkv[:, :qn + 2 * kn]
@@ -340,6 +362,11 @@ class PagedAttention(PagedSoftmaxCore, Mixer):
             ops.conv_silu(qkv, mixed, self.w_conv, None, ws.get("attn.no_state", (1, 1), torch.float32), ctx.token_seg,
                           ctx.seg_slot, ctx.seg_q_start, activation=False)
             qkv = mixed
+        value_source = None
+        if self.value_mix == "source":
+            ctx.shared["attention.values"] = qkv[:, qn + kn:]
+        elif self.value_mix:
+            value_source = ctx.shared["attention.values"]
         q = ws.get("attn.q", (T, qn), ctx.dtype)
         table = ctx.block_tables[cache.block_table_index]
         cos_sin = self.position.table(ctx.device, ctx.max_positions)
@@ -347,7 +374,8 @@ class PagedAttention(PagedSoftmaxCore, Mixer):
             qkv, q, cache.kv_pages if cache.writes else None, self.w_qnorm, self.w_knorm,
             cos_sin, ctx.token_pos, ctx.token_seg, table, self.nq, self.nkv, self.d,
             self.position.rotary_dim, self.norm_mode, self.norm_plus_one,
-            self.position.interleaved, self.norm_eps, norm_dim=self.dk)
+            self.position.interleaved, self.norm_eps, norm_dim=self.dk, value_first=value_source,
+            value_lambda=self.w_value_mix if value_source is not None else None)
         o = ws.get("attn.o", (T, qn), ctx.dtype)
         self.attend(ctx, q, o, cache.kv_pages, table)
         if self.gate == "head":

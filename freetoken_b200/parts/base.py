@@ -143,6 +143,9 @@ class StepContext:
     # when set, parts may leave measurements here (the benchmark counts the
     # experts a step touched); never set on the serving path
     probe: Optional[Dict[str, Any]] = None
+    # what a layer leaves for layers that run after it in the same step (values that later layers
+    # blend in), by a name both know; rows in workspace buffers of their own
+    shared: Dict[str, Any] = field(default_factory=dict)
 
     @property
     def num_segments(self) -> int:
@@ -257,6 +260,11 @@ class Mixer(Part):
 
     def forward(self, ctx: StepContext, x: torch.Tensor, cache: CacheView) -> torch.Tensor:
         raise NotImplementedError
+
+    def forward_parts(self, ctx: StepContext, x: torch.Tensor, cache: CacheView):
+        """``(rows [T, H] or [T, m, H], scales [m] or None)``: the result as rows that the consumer's kernel
+        scales and adds."""
+        return self.forward(ctx, x, cache), None
 
 
 class FeedForward(Part):

@@ -20,6 +20,16 @@ The two outputs leave the block as ``[T, 2, H]``; the next norm adds them to eac
 other and then to the residual in float32 (``x + (mixer + feed_forward)``).  A
 parallel layer may have no feed-forward; then it returns the mixer's rows alone.
 
+``parallel_norms`` is the parallel layer with a norm for each of the two sublayers, both of the same residual
+row::
+
+    h, g = norm1, norm2 (delta, residual)     # residual += delta; one launch, one mean and variance
+    return mixer(h) + feed_forward(g)         # not added yet (:class:`ops.RoutedRows`)
+
+The mixer's rows (with their scales, where several mixers stand side by side), the routed experts' rows and
+the shared expert's gated row leave the block as they are; the next norm adds them all, in float32, in the
+launch that joins them to the residual.
+
 ``sandwich`` norms every sublayer's output as well as its input and scales it before it
 joins the residual stream::
 
@@ -45,6 +55,7 @@ next such norm folds in::
 
 from __future__ import annotations
 
+from ..csrc import ops
 from .base import Block, register_block
 from .norm import NormedBranch, plain_branch
 
@@ -87,6 +98,32 @@ class ParallelBlock(Block):
         else:
             pair[:, 1].copy_(plain_branch(ctx, self.feed_forward.forward(ctx, h)))
         return pair
+
+
+@register_block("parallel_norms")
+class ParallelNormsBlock(Block):
+    NORM_NAMES = ("mixer", "feed_forward")
+    HAS_FEED_FORWARD = True          # or none: then only the mixer's norm
+
+    @classmethod
+    def check_parts(cls, prefix, norm_names, has_feed_forward) -> None:
+        want = cls.NORM_NAMES if has_feed_forward else cls.NORM_NAMES[:1]
+        if sorted(norm_names) != sorted(want):
+            raise ValueError(f"layer '{prefix}': a parallel block with norms of its own {'with' if has_feed_forward else 'without'} "
+                             f"feed-forward has the norms {list(want)}, the layer lists {sorted(norm_names)}")
+
+    def forward(self, ctx, delta, residual, cache):
+        if self.feed_forward is None:
+            h = self.norms["mixer"].forward(ctx, delta, residual)
+            rows, scale = self.mixer.forward_parts(ctx, h, cache)
+            return ops.RoutedRows(rows, scale=scale)
+        h, g = self.norms["mixer"].forward_pair(ctx, delta, residual, self.norms["feed_forward"])
+        rows, scale = self.mixer.forward_parts(ctx, h, cache)
+        out = self.feed_forward.forward(ctx, g)
+        if not isinstance(out, ops.RoutedRows):
+            out = ops.RoutedRows(out)
+        out.beside, out.beside_scale = rows, scale
+        return out
 
 
 @register_block("sandwich")

@@ -56,7 +56,8 @@ class MixerSum(Mixer):
     def libraries(self, dtype):
         return ["rowwise"] + [lib for m in self.members for lib in m.libraries(dtype)]
 
-    def forward(self, ctx: StepContext, x: torch.Tensor, cache: CacheView, out=None) -> torch.Tensor:
+    def forward_parts(self, ctx: StepContext, x: torch.Tensor, cache: CacheView):
+        """``(rows [T, members, H], scales)`` before they are added: for a consumer that adds rows anyway."""
         T, n = x.shape[0], len(self.members)
         rows = ctx.workspace.get("mixer_sum.rows", (T, n, self.hidden), ctx.dtype)
         for j, (member, view) in enumerate(zip(self.members, cache.members)):
@@ -64,6 +65,11 @@ class MixerSum(Mixer):
                 member.forward(ctx, x, view, out=rows[:, j])
             else:
                 rows[:, j].copy_(member.forward(ctx, x, view))
+        return rows, self.scale_tensor
+
+    def forward(self, ctx: StepContext, x: torch.Tensor, cache: CacheView, out=None) -> torch.Tensor:
+        T = x.shape[0]
+        rows, _ = self.forward_parts(ctx, x, cache)
         if out is None:
             out = ctx.workspace.get("mixer_sum.out", (T, self.hidden), ctx.dtype)
         if not out.is_contiguous():

@@ -29,15 +29,19 @@ def linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor,
     names ``f`` (one of ``ops.ACTIVATIONS``; ``None``: the product itself): the weight-streaming
     kernel applies it to its float32 accumulator, behind the other products it is a launch
     of its own on the stored result.  ``bias`` (float32 ``[N]``; not together with an
-    activation) is added to the product: by the library product itself where that runs (its
-    float32 accumulator plus the bias, rounded once), by a launch of its own elsewhere."""
+    activation) is added to the product: by the library product or the weight-streaming kernel itself
+    where those run (their float32 accumulator plus the bias, rounded once), by a launch of its own
+    elsewhere."""
     if bias is not None:
         if activation is not None:
             raise ValueError("linear: a bias and an activation together are not offered")
         rows = x.shape[0]
+        if (x.dtype == torch.bfloat16 and weight.dtype == torch.bfloat16 and rows <= SKINNY_ROWS
+                and ops.skinny_gemm_takes(x, weight, out)):
+            ops.skinny_gemm(x, weight, out, rows_per_pass=ops.pass_rows(rows), bias=bias)
+            return out
         if (x.dtype == torch.bfloat16 and weight.dtype == torch.bfloat16 and out.dtype == torch.bfloat16
-                and out.is_contiguous()
-                and not (rows <= SKINNY_ROWS and ops.skinny_gemm_takes(x, weight, out))):
+                and out.is_contiguous()):
             torch.addmm(_bias_as(bias, torch.bfloat16), x, weight.t(), out=out)
             return out
         linear(x, weight, out)
@@ -66,6 +70,29 @@ def linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor,
             ops.skinny_gemm(x, weight, out, rows_per_pass=32)
             return out
     ops.gemm_rows(x, weight, out)
+    return out
+
+
+def few_rows_glu(x: torch.Tensor, gate_up: torch.Tensor, act: str) -> bool:
+    """Whether a gated pair ``f(Wgate x) * (Wup x)`` of few rows runs as one launch of the weight-streaming kernel."""
+    return (x.dtype == torch.bfloat16 and gate_up.dtype == torch.bfloat16 and x.shape[0] <= SKINNY_ROWS
+            and act in ops.GLU_ACTS and ops.skinny_gemm_takes(x, gate_up, x))
+
+
+def grouped(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """``out[g] = x[g] @ weight[g]^T`` for several matrices of one shape: ``x`` ``[G, T, K]``, ``weight`` ``[G, N,
+    K]``, ``out`` ``[G, T, N]``, all dense.  Few rows: one launch of the weight-streaming kernel over all groups;
+    many: one batched library product; float32: the CUDA-core kernel, group by group."""
+    G, T, K = x.shape
+    if x.dtype == torch.bfloat16 and weight.dtype == torch.bfloat16:
+        rows, flat = x.view(G * T, K), out.view(G * T, out.shape[2])
+        if T <= SKINNY_ROWS and ops.skinny_gemm_takes(rows, weight, flat):
+            ops.skinny_gemm(rows, weight, flat, group_rows=T, rows_per_pass=ops.pass_rows(T))
+            return out
+        torch.bmm(x, weight.transpose(1, 2), out=out)
+        return out
+    for g in range(G):
+        linear(x[g], weight[g], out[g])
     return out
 
 

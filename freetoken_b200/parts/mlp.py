@@ -70,6 +70,14 @@ class DenseMLP(FeedForward):
         ws = ctx.workspace
         if self.gated:
             # one product against [gate; up], then f(gate) * up in float32
+            if linear.few_rows_glu(x, self.w_up, self.act):
+                # decode rows: both halves and f(gate) * up in the weight-streaming kernel
+                mid = ws.get("mlp.mid", (T, self.inter), ctx.dtype)
+                ops.skinny_gemm(x, self.w_up, mid, glu=True, act=self.act, act_alpha=self.act_alpha,
+                                act_limit=self.act_limit, rows_per_pass=ops.pass_rows(T))
+                if out is None:
+                    out = ws.get("mlp.y", (T, self.hidden), ctx.dtype)
+                return linear.linear(mid, self.w_down, out)
             both = linear.linear(x, self.w_up, ws.get("mlp.gate_up", (T, 2 * self.inter), ctx.dtype))
             mid = ws.get("mlp.mid", (T, self.inter), ctx.dtype)
             ops.glu_rows(both, mid, self.act, self.act_alpha, self.act_limit)

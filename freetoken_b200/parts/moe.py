@@ -14,7 +14,8 @@ accumulator; ``y = sum over the k routes`` in float32, slot order.
 Two options no model of the reference has: ``identity`` - the last outputs of the router stand for
 experts without weights that hand the input back, times the route's weight (their routes are sorted
 behind all others and no product touches them) - and ``shared``, a gated feed-forward every token
-passes, added.  With either the result is :class:`ops.RoutedRows`: the consumer's kernel adds the
+passes, added (``shared_gate``: times ``sigmoid(w h)``, one number per token, whose row rides behind the
+router's in one float32 product).  With either the result is :class:`ops.RoutedRows`: the consumer's kernel adds the
 routed rows, the handed-back input and the shared row in float32, in one pass.
 Activation ``silu`` or ``swigluoai``
 (python/freetoken/kernel/triton/activation.py:96-107).
@@ -69,10 +70,12 @@ class RoutedExperts(FeedForward):
     (router, bias, gate_up, down: model-side names below the scope; gate, up,
     down_each: per-expert checkpoint names with ``{e}``).  ``groups`` and ``keep_groups``
     (default 1, 1: no groups): the experts form ``groups`` equal groups of neighbours, a group's
-    value is the sum of its two largest choice scores (score plus bias), and only experts of the
-    ``keep_groups`` best groups can be chosen.  ``identity`` (default 0): so many router outputs behind
+    value is the sum of its two largest choice scores (score plus bias; ``group_top`` 1: the largest), and
+    only experts of the ``keep_groups`` best groups can be chosen.  ``identity`` (default 0): so many router outputs behind
     the ``num_experts`` experts' hand the input back.  ``shared`` (a PartSpec of a feed-forward, or
-    None): one that runs for every token beside the routed experts."""
+    None): one that runs for every token beside the routed experts; ``shared_gate`` (default False) gates
+    it per token (``checkpoint_names`` then also has shared_gate, ``[1, hidden]``, and router_gate, the name
+    of the merged matrix the model keeps)."""
 
     graph_capturable = True
 
@@ -100,7 +103,13 @@ class RoutedExperts(FeedForward):
                 or self.keep_groups * (self.outputs // self.groups) < self.k or self.groups > 256):
             raise ValueError(f"{self.groups} groups of which {self.keep_groups} are kept do not fit "
                              f"{self.outputs} experts, top-{self.k}")
+        self.group_top = int(p.get("group_top", 2))
+        if self.group_top not in (1, 2):
+            raise ValueError("a group's value is made of its largest one or two choice scores")
         self.shared = None
+        self.shared_gate = bool(p.get("shared_gate", False))
+        if self.shared_gate and (p.get("shared") is None or self.identity):
+            raise ValueError("a gate on the shared feed-forward needs one (and no identity experts beside it)")
         if p.get("shared") is not None:
             self.shared = FEED_FORWARDS.get(p["shared"].kind)(p["shared"], prefix)
             if not self.shared.writes_into_out:
@@ -111,6 +120,10 @@ class RoutedExperts(FeedForward):
         self.n_bias = f"{self.scope}.{names['bias']}"
         self.n_gate_up = f"{self.scope}.{names['gate_up']}"
         self.n_down = f"{self.scope}.{names['down']}"
+        if self.shared_gate:
+            self.n_shared_gate = f"{self.scope}.{names['shared_gate']}"
+            self.n_router_gate = f"{self.scope}.{names['router_gate']}"
+        self.logit_rows = self.outputs + (1 if self.shared_gate else 0)
         self._each = {key: f"{self.scope}.{names[key]}" for key in ("gate", "up", "down_each")}
         self.w_router = self.w_router_terms = self.w_bias = self.w_gate_up = self.w_down = None
 
@@ -123,8 +136,13 @@ class RoutedExperts(FeedForward):
             Cat((Name(self._each["gate"].format(e=e), (I, H)),
                  Name(self._each["up"].format(e=e), (I, H))), 0) for e in range(E)))
         down = Stack(tuple(Name(self._each["down_each"].format(e=e), (H, I)) for e in range(E)))
+        router = TensorSpec(self.n_router, (self.outputs, H), role="small32", keep_float32_in_file=True)
+        if self.shared_gate:
+            router = TensorSpec(self.n_router_gate, (self.outputs + 1, H), role="small32", keep_float32_in_file=True,
+                                sources=(Cat((Name(self.n_router, (self.outputs, H)),
+                                              Name(self.n_shared_gate, (1, H))), 0),))
         return [
-            TensorSpec(self.n_router, (self.outputs, H), role="small32", keep_float32_in_file=True),
+            router,
             TensorSpec(self.n_bias, (self.outputs,), role="small32", keep_float32_in_file=True,
                        init=Init(0.0, 0.01 if self.use_bias else 0.0), tag="router_bias",
                        optional=not self.use_bias),
@@ -133,7 +151,7 @@ class RoutedExperts(FeedForward):
         ] + (self.shared.tensor_specs() if self.shared is not None else [])
 
     def bind(self, tensors: Dict[str, torch.Tensor], dtype) -> None:
-        self.w_router = tensors[self.n_router]
+        self.w_router = tensors[self.n_router_gate if self.shared_gate else self.n_router]
         self.w_router_terms = bf16_terms(self.w_router) if dtype == torch.bfloat16 else None
         # The bias is part of the routing whenever the checkpoint carries it: the
         # reference's block always adds it (python/freetoken/models/minimax_m3/moe.py:75,
@@ -157,7 +175,7 @@ class RoutedExperts(FeedForward):
         whether that was done here (a handful of tokens: one launch for both)."""
         T = x.shape[0]
         ws = ctx.workspace
-        logits = ws.get("moe.logits", (T, self.outputs), torch.float32)
+        logits = ws.get("moe.logits", (T, self.logit_rows), torch.float32)
         terms = 1
         if ctx.dtype == torch.bfloat16 and T <= ROUTER_SMALL_T and ops.router_logits_takes(x, self.w_router):
             ops.router_logits(x, self.w_router, logits)
@@ -166,18 +184,20 @@ class RoutedExperts(FeedForward):
                                                torch.float32)):
             # many rows: tensor-core products of the bfloat16 activations with the exact
             # bfloat16 terms of the float32 router weight; the terms are summed by the selection
-            terms = self.w_router_terms.shape[0] // self.outputs
+            terms = self.w_router_terms.shape[0] // self.logit_rows
             logits = ws.get("moe.logit_terms", (T, self.w_router_terms.shape[0]), torch.float32)
         else:
             ops.gemm_rows(x, self.w_router, logits)
         ids = ws.get("moe.ids", (T, self.k), torch.int32)
         weights = ws.get("moe.weights", (T, self.k), torch.float32)
+        gate = ws.get("moe.shared_gate", (T,), torch.float32) if self.shared_gate else None
         if sort_into is not None and ops.route_small_takes(T, self.outputs, self.k):
             ops.route_small(logits, self.w_bias, ids, weights, *sort_into, self.k, self.softmax,
-                            self.renorm, self.scale, terms, self.groups, self.keep_groups, busy_of=self.E)
+                            self.renorm, self.scale, terms, self.groups, self.keep_groups, busy_of=self.E,
+                            group_top=self.group_top, tail=gate)
             return ids, weights, True
         ops.router_select(logits, self.w_bias, ids, weights, self.k, self.softmax, self.renorm,
-                          self.scale, terms, self.groups, self.keep_groups)
+                          self.scale, terms, self.groups, self.keep_groups, self.group_top, gate)
         return (ids, weights) if sort_into is None else (ids, weights, False)
 
     def forward(self, ctx: StepContext, x: torch.Tensor):
@@ -214,7 +234,8 @@ class RoutedExperts(FeedForward):
         if self.shared is not None:
             extra = self.shared.forward(ctx, x, out=ws.get("moe.shared", (T, self.hidden), ctx.dtype))
         if not self.identity:
-            return ops.RoutedRows(parts, extra=extra)
+            gate = ws.get("moe.shared_gate", (T,), torch.float32) if self.shared_gate else None
+            return ops.RoutedRows(parts, extra=extra, extra_gate=gate)
         return ops.RoutedRows(parts, ids, weights, self.E, x, extra)
 
     def experts(self, ctx, x, mid, parts, offsets, active, sorted_route, sorted_token, route_weight, R):

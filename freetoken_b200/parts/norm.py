@@ -120,6 +120,65 @@ class PendingBranch:
         self.y, self.mix, self.out = y, mix, out
 
 
+@register_norm("layer_norm")
+class LayerNorm(Norm):
+    """Layer norm with the residual add folded in: the pending branch joins, then ``(x - mean) / sqrt(variance +
+    eps) * weight [+ bias]``, the variance being the mean of the squared deviations.  params: ``size``, ``eps``,
+    ``tensor`` (the weight's name below the prefix), ``bias_tensor`` (None: no bias), ``factor`` (default 1): a
+    constant on the result - in front of a head, a factor on the logits that costs no pass over them; it is
+    multiplied into weight and bias at binding, in float32."""
+
+    graph_capturable = True
+
+    def __init__(self, spec, prefix):
+        super().__init__(spec, prefix)
+        p = spec.params
+        self.size = int(p["size"])
+        self.eps = float(p["eps"])
+        self.factor = float(p.get("factor", 1.0))
+        self.weight_name = self.name(p["tensor"])
+        self.bias_name = self.name(p["bias_tensor"]) if p.get("bias_tensor") else None
+        self.weight = self.bias = None
+
+    def tensor_specs(self) -> List[TensorSpec]:
+        specs = [TensorSpec(self.weight_name, (self.size,), role="small32", init=Init(mean=1.0, std=0.0), tag="norm")]
+        if self.bias_name:
+            specs.append(TensorSpec(self.bias_name, (self.size,), role="small32", init=Init(0.0, 0.02), tag="bias"))
+        return specs
+
+    def bind(self, tensors: Dict[str, torch.Tensor], dtype) -> None:
+        self.weight = tensors[self.weight_name]
+        self.bias = tensors[self.bias_name] if self.bias_name else None
+        if self.factor != 1.0:
+            self.weight = self.weight * self.factor
+            self.bias = self.bias * self.factor if self.bias is not None else None
+
+    def libraries(self, dtype) -> List[str]:
+        return ["rowwise"]
+
+    def _join(self, ctx: StepContext, delta, residual: torch.Tensor):
+        """What is left to join: a branch with a norm of its own joins by a launch of its own."""
+        if isinstance(delta, PendingBranch):
+            raise ValueError("a branch with connection weights joins several streams, not the plain residual")
+        if isinstance(delta, NormedBranch):
+            delta.norm.add_normed(ctx, delta.y, residual, delta.mult)
+            return None
+        return delta
+
+    def forward(self, ctx: StepContext, delta, residual: torch.Tensor) -> torch.Tensor:
+        out = ctx.workspace.get("norm.out", residual.shape, ctx.dtype)
+        ops.join_layer_norm(self._join(ctx, delta, residual), residual, self.weight, self.eps, out, self.bias)
+        return out
+
+    def forward_pair(self, ctx: StepContext, delta, residual: torch.Tensor, other: "LayerNorm"):
+        """``(this norm's rows, other's rows)`` of the same new residual rows, in one launch."""
+        out = ctx.workspace.get("norm.out", residual.shape, ctx.dtype)
+        out2 = ctx.workspace.get("norm.out2", residual.shape, ctx.dtype)
+        ops.join_layer_norm(self._join(ctx, delta, residual), residual, self.weight, self.eps, out, self.bias,
+                            other.weight, other.eps, out2, other.bias)
+        return out, out2
+
+
 @register_norm("hyper_norm")
 class HyperNorm(Norm):
     """The norm in front of a sublayer of a model with several residual streams

@@ -22,6 +22,11 @@ head's state, ``x``/``v`` its input row of ``head_dim`` values:
   rotated by their position, no convolution; ``o`` is RMS-normed per head without a weight and
   gated by ``silu``.
 
+* ``time_mixing`` (the recurrence of RWKV with a decay made from the input): every projection reads a mix
+  of its own of the token's and the previous token's input, ``h + (h' - h) mu``; ``w = exp(-exp(W_w2
+  tanh(W_w1 mix) + w0))`` per key channel, ``o = (S + diag(u) k v^T)^T r``, then ``S <- diag(w) S + k v^T``; each
+  head's ``o`` is RMS-normed, the row gated by ``silu``.  The previous token's input is part of the state.
+
 A request's state is one float32 row ``[convolution inputs | recurrent state]`` in
 its slot (:class:`StateNeed`); the kernels take segments of any length, so a
 prompt portion and a decoded token run the same code.  The reference keeps such
@@ -36,7 +41,7 @@ import torch
 
 from ..cache.manager import StateNeed
 from ..csrc import ops
-from ..weights.spec import Cat, Init, Name, TensorSpec
+from ..weights.spec import Cat, Init, Name, Stack, TensorSpec
 from . import linear
 from .base import POSITIONS, CacheView, Mixer, StepContext, register_mixer
 
@@ -338,4 +343,83 @@ class Retention(_Recurrent):
         ops.gated_norm(o, proj[:, 2 * kd + inner:], self.ones, gated, self.heads, self.eps, gate_first=False)
         if out is None:
             out = ws.get("retention.out", (T, self.hidden), ctx.dtype)
+        return linear.linear(gated, w["o"], out)
+
+
+@register_mixer("time_mixing")
+class TimeMixing(Mixer):
+    """params: ``hidden_size, heads, key_dim, head_dim, low_rank`` (the width of the middle of the decay's
+    two-step projection), ``norm_eps``, ``scope`` and ``names`` (mu_r, mu_k, mu_v, mu_g, mu_w: the mixes; r, k, v,
+    gate: projections; decay_down, decay_up: the decay's two steps; w0, u, norm, o; mu and rkvg: the merged
+    mixes and projections the model keeps).  ``r, k, v`` and ``gate`` rows have one width, so ``key_dim`` must equal
+    ``head_dim``; ``norm`` has one entry per value of the concatenated heads."""
+
+    graph_capturable = True
+    writes_into_out = True
+
+    MIXES = ("r", "k", "v", "g", "w")
+
+    def __init__(self, spec, prefix):
+        super().__init__(spec, prefix)
+        p = spec.params
+        self.hidden = int(p["hidden_size"])
+        self.heads = int(p["heads"])
+        self.D = int(p["key_dim"])
+        self.P = int(p["head_dim"])
+        self.low = int(p["low_rank"])
+        self.eps = float(p["norm_eps"])
+        if self.D != self.P or self.D > 256 or self.low < 1:
+            raise ValueError("time_mixing: key_dim must equal head_dim (at most 256), low_rank must be positive")
+        self.inner = self.heads * self.P
+        self.state_values = self.heads * self.D * self.P
+        scope = self.name(p["scope"])
+        self.names = {key: f"{scope}.{local}" for key, local in p["names"].items()}
+        self.w: Dict[str, torch.Tensor] = {}
+
+    def cache_need(self):
+        return StateNeed((self.hidden + self.state_values,), "float32")
+
+    def tensor_specs(self) -> List[TensorSpec]:
+        n, H, inner = self.names, self.hidden, self.inner
+        small = dict(role="small32", tag="recurrent")
+        return [
+            TensorSpec(n["mu"], (len(self.MIXES) * H,), init=Init(0.5, 0.2), sources=(Cat(tuple(
+                Name(n["mu_" + m], (H,)) for m in self.MIXES), 0),), **small),
+            TensorSpec(n["rkvg"], (4, inner, H), sources=(Stack(tuple(
+                Name(n[key], (inner, H)) for key in ("r", "k", "v", "gate"))),)),
+            TensorSpec(n["decay_down"], (self.low, H)),
+            TensorSpec(n["decay_up"], (inner, self.low), init=Init(0.0, 0.2)),
+            TensorSpec(n["w0"], (inner,), init=Init(-1.0, 1.0), **small),
+            TensorSpec(n["u"], (self.heads, self.D), init=Init(0.5, 0.3), **small),
+            TensorSpec(n["norm"], (inner,), role="small32", init=Init(1.0, 0.0), tag="norm"),
+            TensorSpec(n["o"], (H, inner), tag="residual_out"),
+        ]
+
+    def bind(self, tensors, dtype) -> None:
+        self.w = {key: tensors[self.names[key]]
+                  for key in ("mu", "rkvg", "decay_down", "decay_up", "w0", "u", "norm", "o")}
+        self.w["mu"] = self.w["mu"].view(len(self.MIXES), self.hidden)
+
+    def libraries(self, dtype) -> List[str]:
+        return ["time_mixing", "recurrent", "rowwise"] + linear.libraries(dtype)
+
+    def forward(self, ctx: StepContext, x: torch.Tensor, cache: CacheView, out=None) -> torch.Tensor:
+        T, ws, w = x.shape[0], ctx.workspace, self.w
+        inner = self.inner
+        if cache.state is None or not cache.writes:
+            raise ValueError("TimeMixing needs state slots of its own")
+        previous, state = cache.state[:, :self.hidden], cache.state[:, self.hidden:]
+        mixed = ws.get("tmix.mixed", (len(self.MIXES), T, self.hidden), ctx.dtype)
+        ops.token_shift(x, w["mu"], mixed, previous, ctx.token_seg, ctx.seg_slot, ctx.seg_q_start)
+        rkvg = linear.grouped(mixed[:4], w["rkvg"], ws.get("tmix.rkvg", (4, T, inner), ctx.dtype))
+        low = linear.linear(mixed[4], w["decay_down"], ws.get("tmix.low", (T, self.low), ctx.dtype), activation="tanh")
+        # the decay's second step leaves its float32 accumulator: both exponentials follow in float32
+        decay = linear.linear(low, w["decay_up"], ws.get("tmix.decay", (T, inner), torch.float32))
+        o = ws.get("tmix.o", (T, inner), torch.float32)
+        ops.time_mixing_scan(rkvg[0], rkvg[1], rkvg[2], decay, w["w0"], w["u"], state, o, ctx.seg_slot, ctx.seg_q_start,
+                             self.heads, self.P, self.D)
+        gated = ws.get("tmix.gated", (T, inner), ctx.dtype)
+        ops.gated_norm(o, rkvg[3], w["norm"], gated, self.heads, self.eps, gate_first=False)
+        if out is None:
+            out = ws.get("tmix.out", (T, self.hidden), ctx.dtype)
         return linear.linear(gated, w["o"], out)

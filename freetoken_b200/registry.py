@@ -150,3 +150,13 @@ def _load_builtin() -> None:
             config_to_dict=lambda cfg: cfg.to_dict(),
         ),
     )
+    from .config import besuzen
+    register_architecture(
+        Architecture(
+            name=besuzen.ARCHITECTURE,
+            read_config=besuzen.BesuzenConfig.from_dict,
+            build_plan=besuzen.build_plan,
+            config_to_dict=lambda cfg: cfg.to_dict(),
+            sizes_from_tensors=besuzen.sizes_from_tensors,
+        ),
+    )
