@@ -10,7 +10,8 @@ same for the Tonapel decoder (freetoken_b200/tonapel_bench.py), ``--design nirel
 decoder beside the Tonapel decoder at equal size (freetoken_b200/nirelix_bench.py), ``--design mezapel``
 the Mezapel decoder beside the MiniMax-M3 decoder at equal size (freetoken_b200/mezapel_bench.py),
 ``--design dizatar`` the Dizatar decoder beside a Nirelix decoder of latent-attention layers at equal size
-(freetoken_b200/dizatar_bench.py).
+(freetoken_b200/dizatar_bench.py), ``--design besuzen`` the Besuzen decoder beside the Tonapel decoder at
+equal size (freetoken_b200/besuzen_bench.py).
 """
 import os
 import sys

@@ -346,10 +346,13 @@ __device__ __forceinline__ float4 branch_at4(const BranchArgs& b, int t, int H, 
   }
   if (b.beside) {
     const AT* other = (const AT*)b.beside + (size_t)t * b.kb * H + 4 * gi;
-    for (int j = 0; j < b.kb; ++j) {
-      const float4 v = load4f(other + (size_t)j * H);
-      const float s = b.beside_scale ? b.beside_scale[j] : 1.f;
-      y.x = fmaf(s, v.x, y.x); y.y = fmaf(s, v.y, y.y); y.z = fmaf(s, v.z, y.z); y.w = fmaf(s, v.w, y.w);
+    for (int j0 = 0; j0 < b.kb; j0 += 2) {
+      const bool second = j0 + 1 < b.kb;
+      const float4 v0 = load4f(other + (size_t)j0 * H), v1 = second ? load4f(other + (size_t)(j0 + 1) * H) : zero;
+      const float s0 = b.beside_scale ? b.beside_scale[j0] : 1.f;
+      const float s1 = b.beside_scale && second ? b.beside_scale[j0 + 1] : 1.f;
+      y.x = fmaf(s0, v0.x, y.x); y.y = fmaf(s0, v0.y, y.y); y.z = fmaf(s0, v0.z, y.z); y.w = fmaf(s0, v0.w, y.w);
+      y.x = fmaf(s1, v1.x, y.x); y.y = fmaf(s1, v1.y, y.y); y.z = fmaf(s1, v1.z, y.z); y.w = fmaf(s1, v1.w, y.w);
     }
   }
   if (back != 0.f) h = load4f((const AT*)b.source + (size_t)t * H + 4 * gi);
@@ -542,7 +545,8 @@ struct JoinNormArgs {
   float eps1, eps2;
 };
 
-template <typename AT, int KEEP, int THREADS>
+// EAGER (few tokens): the weights are fetched with the rows, before the sums.
+template <typename AT, int KEEP, int THREADS, bool EAGER = false>
 __global__ void __launch_bounds__(THREADS) join_layer_norm_kernel(JoinNormArgs a) {
   extern __shared__ float row[];
   __shared__ float scratch[33];
@@ -554,9 +558,20 @@ __global__ void __launch_bounds__(THREADS) join_layer_norm_kernel(JoinNormArgs a
   const bool two = a.w2 != nullptr;
   float sum = 0.f, sq = 0.f;
   if constexpr (KEEP > 0) {
-    float4 x[KEEP];
+    float4 x[KEEP], e1[EAGER ? KEEP : 1], e2[EAGER ? KEEP : 1];
     const int groups = H >> 2;
     float back = 0.f;
+    if constexpr (EAGER) {
+#pragma unroll
+      for (int j = 0; j < KEEP; ++j) {
+        const int gi = threadIdx.x + j * THREADS;
+        e1[j] = e2[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (gi < groups) {
+          e1[j] = load4f(a.w1 + 4 * gi);
+          if (two) e2[j] = load4f(a.w2 + 4 * gi);
+        }
+      }
+    }
     const unsigned slots = a.b.rows ? branch_slots(a.b, t, back) : 0u;
 #pragma unroll
     for (int j = 0; j < KEEP; ++j) {
@@ -583,13 +598,13 @@ __global__ void __launch_bounds__(THREADS) join_layer_norm_kernel(JoinNormArgs a
       }
     }
     const float var = block_sum(sq, scratch) / (float)H;
-    auto write = [&](AT* o, const float* w, const float* b, float eps) {
+    auto write = [&](AT* o, const float* w, const float4* eager, const float* b, float eps) {
       const float inv = 1.f / sqrtf(var + eps);
 #pragma unroll
       for (int j = 0; j < KEEP; ++j) {
         const int gi = threadIdx.x + j * THREADS;
         if (gi < groups) {
-          const float4 wv = load4f(w + 4 * gi);
+          const float4 wv = EAGER ? eager[EAGER ? j : 0] : load4f(w + 4 * gi);
           float4 v = make_float4(x[j].x * inv * wv.x, x[j].y * inv * wv.y, x[j].z * inv * wv.z, x[j].w * inv * wv.w);
           if (b) {
             const float4 bv = load4f(b + 4 * gi);
@@ -599,8 +614,8 @@ __global__ void __launch_bounds__(THREADS) join_layer_norm_kernel(JoinNormArgs a
         }
       }
     };
-    write(o1, a.w1, a.b1, a.eps1);
-    if (two) write(o2, a.w2, a.b2, a.eps2);
+    write(o1, a.w1, e1, a.b1, a.eps1);
+    if (two) write(o2, a.w2, e2, a.b2, a.eps2);
   } else {
     for (int i = threadIdx.x; i < H; i += THREADS) {
       float v = r[i];
@@ -1231,10 +1246,15 @@ int ft_join_layer_norm(const BranchArgs* branch, float* residual, const float* w
                    !((uintptr_t)w1 & 15) && !((uintptr_t)b1 & 15) && !((uintptr_t)w2 & 15) && !((uintptr_t)b2 & 15) &&
                    !((uintptr_t)out1 & 15) && !((uintptr_t)out2 & 15);
   const dim3 g(T), th(256);
-  if (vec && H <= 1024) { FT_DISPATCH(dtype, AT, (launch_pdl(join_layer_norm_kernel<AT, 1, 256>, g, th, 0, stream, a))); }
+  const bool eager = vec && T <= 256;      // the threads a row gets depend on its width alone: so do its sums
+  if (eager && H <= 1024) { FT_DISPATCH(dtype, AT, (launch_pdl(join_layer_norm_kernel<AT, 1, 256, true>, g, th, 0, stream, a))); }
+  else if (eager && H <= 2048) { FT_DISPATCH(dtype, AT, (launch_pdl(join_layer_norm_kernel<AT, 2, 256, true>, g, th, 0, stream, a))); }
+  else if (eager && H <= 4096) { FT_DISPATCH(dtype, AT, (launch_pdl(join_layer_norm_kernel<AT, 2, 512, true>, g, dim3(512), 0, stream, a))); }
+  else if (eager) { FT_DISPATCH(dtype, AT, (launch_pdl(join_layer_norm_kernel<AT, 4, 512, true>, g, dim3(512), 0, stream, a))); }
+  else if (vec && H <= 1024) { FT_DISPATCH(dtype, AT, (launch_pdl(join_layer_norm_kernel<AT, 1, 256>, g, th, 0, stream, a))); }
   else if (vec && H <= 2048) { FT_DISPATCH(dtype, AT, (launch_pdl(join_layer_norm_kernel<AT, 2, 256>, g, th, 0, stream, a))); }
-  else if (vec && H <= 4096) { FT_DISPATCH(dtype, AT, (launch_pdl(join_layer_norm_kernel<AT, 4, 256>, g, th, 0, stream, a))); }
-  else if (vec) { FT_DISPATCH(dtype, AT, (launch_pdl(join_layer_norm_kernel<AT, 8, 256>, g, th, 0, stream, a))); }
+  else if (vec && H <= 4096) { FT_DISPATCH(dtype, AT, (launch_pdl(join_layer_norm_kernel<AT, 2, 512>, g, dim3(512), 0, stream, a))); }
+  else if (vec) { FT_DISPATCH(dtype, AT, (launch_pdl(join_layer_norm_kernel<AT, 4, 512>, g, dim3(512), 0, stream, a))); }
   else {
     FT_DISPATCH(dtype, AT, (launch_pdl(join_layer_norm_kernel<AT, 0, 256>, g, th, (size_t)H * sizeof(float), stream, a)));
   }

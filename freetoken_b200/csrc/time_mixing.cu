@@ -109,18 +109,17 @@ __global__ void __launch_bounds__(128) token_shift_kernel(ShiftArgs a) {
 }
 
 // ------------------------------------------------------------------------- scan
-// A column of a head's state is shared by 8 lanes; lane l holds rows (8 j + l) 4 .. + 3 for j < RPL / 4, so that
-// 8 lanes read 128 consecutive bytes of r, k, w (and of the state, which is kept value by value: [P][D]).  A
-// warp owns 4 columns, a block TM_COLS.  Tokens come in chunks of 8: every thread fetches its share of the
-// NEXT chunk into registers while the block works through the current one in shared memory and puts it into the
-// other of two buffers afterwards: one barrier a chunk.  The decay's exponentials and the bonus u . (r k) are
-// formed on the way into shared memory.  The read-out's partial sums of the 8 tokens are added over the 8 lanes
-// together, each lane ending with the total of one token: 7 shuffles a chunk.
-constexpr int TM_WARPS = 4;
+// A column of a head's state is shared by LPC lanes; lane l holds rows (LPC j + l) 4 .. + 3 for j < RPL / 4, so
+// that the lanes read consecutive pieces of r, k, w (and of the state, which is kept value by value: [P][D]).  A
+// warp owns 32 / LPC columns, a block of 8 warps 256 / LPC.  Tokens come in chunks of 8: every warp fetches one
+// token of the NEXT chunk into registers while the block works through the current chunk in shared memory and puts
+// it into the other of two buffers afterwards: one barrier a chunk.  The decay's exponentials and the bonus
+// u . (r k) are formed on the way into shared memory.  The read-out's partial sums of the 8 tokens are added over the
+// lanes together, each lane ending with the total of one token: 8 shuffles a chunk.
+constexpr int TM_WARPS = 8;
 constexpr int TM_THREADS = 32 * TM_WARPS;
-constexpr int TM_COLS = 4 * TM_WARPS;
 constexpr int TM_CHUNK = 8;
-static_assert(TM_CHUNK * TM_COLS == TM_THREADS && TM_CHUNK == 2 * TM_WARPS, "a thread stages one value a chunk");
+static_assert(TM_CHUNK == TM_WARPS, "a warp stages a token");
 
 struct TimeMixArgs {
   const void *r, *k, *v;   // row t: r + t * ld, head h's D values at h * D (v: h * P)
@@ -134,22 +133,25 @@ struct TimeMixArgs {
   int heads, P, D, vec;    // vec: state rows may be read in 16-byte pieces
 };
 
-__host__ __device__ constexpr int time_mix_buffer(int RPL) { return TM_CHUNK * (3 * 8 * RPL + TM_COLS + 1); }
+constexpr int time_mix_buffer(int RPL, int LPC) { return TM_CHUNK * (3 * LPC * RPL + TM_THREADS / LPC + 1); }
 
-template <typename AT, int RPL>
+template <typename AT, int RPL, int LPC>
 __global__ void __launch_bounds__(TM_THREADS) time_mixing_kernel(TimeMixArgs a) {
-  constexpr int DP = 8 * RPL;                          // rows, filled up
+  constexpr int DP = LPC * RPL;                        // rows, filled up
   constexpr int NE = DP / 32;                          // channels a lane stages per token
-  constexpr int PER = time_mix_buffer(RPL);
+  constexpr int CPW = 32 / LPC, COLS = TM_WARPS * CPW; // columns of a warp, of a block
+  constexpr int LOG = LPC == 8 ? 3 : 4;
+  constexpr int PER = time_mix_buffer(RPL, LPC);
+  static_assert((LPC == 8 || LPC == 16) && DP % 32 == 0 && TM_CHUNK * COLS <= TM_THREADS, "lanes, rows, columns");
   extern __shared__ __align__(16) float sm[];
   pdl_wait();
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, l = lane & 7;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, l = lane & (LPC - 1);
   const int head = blockIdx.y, seg = blockIdx.z;
   const int D = a.D, P = a.P;
   const int q0 = a.seg_q_start[seg], q1 = a.seg_q_start[seg + 1];
   if (q1 <= q0) return;
-  const int cb = warp * 4 + (lane >> 3);               // this lane's column inside the block
-  const int col = blockIdx.x * TM_COLS + cb;
+  const int cb = warp * CPW + (lane >> LOG);           // this lane's column inside the block
+  const int col = blockIdx.x * COLS + cb;
   float* st = a.state + (size_t)a.seg_slot[seg] * a.slot_stride + ((size_t)head * P + col) * D;
   const AT* rp = (const AT*)a.r + (size_t)head * D;
   const AT* kp = (const AT*)a.k + (size_t)head * D;
@@ -159,7 +161,7 @@ __global__ void __launch_bounds__(TM_THREADS) time_mixing_kernel(TimeMixArgs a) 
   float S[RPL];
 #pragma unroll
   for (int j = 0; j < RPL / 4; ++j) {
-    const int n = (8 * j + l) * 4;
+    const int n = (LPC * j + l) * 4;
     float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
     if (col < P && n < D) {
       if (a.vec) f = *reinterpret_cast<const float4*>(st + n);
@@ -180,25 +182,21 @@ __global__ void __launch_bounds__(TM_THREADS) time_mixing_kernel(TimeMixArgs a) 
     u[e] = n < D ? a.u[(size_t)head * D + n] : 0.f;
   }
 
-  // this warp stages tokens 2 warp and 2 warp + 1 of a chunk, this thread one value of v
-  AT pr[2][NE], pk[2][NE], pv;
-  float pd[2][NE];
-  const int vt = threadIdx.x / TM_COLS, vc = threadIdx.x % TM_COLS;
+  // this warp stages token `warp` of a chunk, the first TM_CHUNK * COLS threads one value of v each
+  AT pr[NE], pk[NE], pv;
+  float pd[NE];
+  const int vt = threadIdx.x / COLS, vc = threadIdx.x % COLS;
   auto fetch = [&](int t0, int nt) {
+    const size_t t = t0 + warp;
 #pragma unroll
-    for (int s = 0; s < 2; ++s) {
-      const int tt = 2 * warp + s;
-      const size_t t = t0 + tt;
-#pragma unroll
-      for (int e = 0; e < NE; ++e) {
-        const int n = lane + 32 * e;
-        const bool in = tt < nt && n < D;
-        pr[s][e] = in ? rp[t * a.ld + n] : from_float<AT>(0.f);
-        pk[s][e] = in ? kp[t * a.ld + n] : from_float<AT>(0.f);
-        pd[s][e] = in ? dp[t * a.ld_decay + n] : 0.f;
-      }
+    for (int e = 0; e < NE; ++e) {
+      const int n = lane + 32 * e;
+      const bool in = warp < nt && n < D;
+      pr[e] = in ? rp[t * a.ld + n] : from_float<AT>(0.f);
+      pk[e] = in ? kp[t * a.ld + n] : from_float<AT>(0.f);
+      pd[e] = in ? dp[t * a.ld_decay + n] : 0.f;
     }
-    const int c = blockIdx.x * TM_COLS + vc;
+    const int c = blockIdx.x * COLS + vc;
     pv = (vt < nt && c < P) ? vp[(size_t)(t0 + vt) * a.ld + c] : from_float<AT>(0.f);
   };
   auto put = [&](float* buf) {
@@ -206,24 +204,20 @@ __global__ void __launch_bounds__(TM_THREADS) time_mixing_kernel(TimeMixArgs a) 
     float* ks = rs + TM_CHUNK * DP;
     float* ws = ks + TM_CHUNK * DP;
     float* vs = ws + TM_CHUNK * DP;
-    float* bs = vs + TM_CHUNK * TM_COLS;
+    float* bs = vs + TM_CHUNK * COLS;
+    float bonus = 0.f;
 #pragma unroll
-    for (int s = 0; s < 2; ++s) {
-      const int tt = 2 * warp + s;
-      float bonus = 0.f;
-#pragma unroll
-      for (int e = 0; e < NE; ++e) {
-        const int n = lane + 32 * e;
-        const float rv = to_float(pr[s][e]), kv = to_float(pk[s][e]);
-        rs[tt * DP + n] = rv;
-        ks[tt * DP + n] = kv;
-        ws[tt * DP + n] = expf(-expf(pd[s][e] + w0[e]));
-        bonus = fmaf(rv * kv, u[e], bonus);
-      }
-      bonus = warp_sum(bonus);
-      if (lane == 0) bs[tt] = bonus;
+    for (int e = 0; e < NE; ++e) {
+      const int n = lane + 32 * e;
+      const float rv = to_float(pr[e]), kv = to_float(pk[e]);
+      rs[warp * DP + n] = rv;
+      ks[warp * DP + n] = kv;
+      ws[warp * DP + n] = expf(-expf(pd[e] + w0[e]));
+      bonus = fmaf(rv * kv, u[e], bonus);
     }
-    vs[threadIdx.x] = to_float(pv);
+    bonus = warp_sum(bonus);
+    if (lane == 0) bs[warp] = bonus;
+    if (vt < TM_CHUNK) vs[threadIdx.x] = to_float(pv);
   };
 
   fetch(q0, min(TM_CHUNK, q1 - q0));
@@ -238,14 +232,14 @@ __global__ void __launch_bounds__(TM_THREADS) time_mixing_kernel(TimeMixArgs a) 
     const float* ks = rs + TM_CHUNK * DP;
     const float* ws = ks + TM_CHUNK * DP;
     const float* vs = ws + TM_CHUNK * DP;
-    const float* bs = vs + TM_CHUNK * TM_COLS;
+    const float* bs = vs + TM_CHUNK * COLS;
     float part[TM_CHUNK];
     auto token = [&](int tt) {
-      const float v = vs[tt * TM_COLS + cb];
+      const float v = vs[tt * COLS + cb];
       float acc = 0.f;
 #pragma unroll
       for (int j = 0; j < RPL / 4; ++j) {
-        const int n = tt * DP + (8 * j + l) * 4;
+        const int n = tt * DP + (LPC * j + l) * 4;
         const float4 r4 = *reinterpret_cast<const float4*>(rs + n);
         const float4 k4 = *reinterpret_cast<const float4*>(ks + n);
         const float4 w4 = *reinterpret_cast<const float4*>(ws + n);
@@ -267,25 +261,29 @@ __global__ void __launch_bounds__(TM_THREADS) time_mixing_kernel(TimeMixArgs a) 
 #pragma unroll
       for (int tt = 0; tt < TM_CHUNK; ++tt) part[tt] = tt < nt ? token(tt) : 0.f;
     }
-    // lane l of a column's 8 ends with token l's total
+    // lane l of a column's ends with the total of token l >> (LOG - 3)
+    int mask = LPC / 2;
 #pragma unroll
     for (int w = TM_CHUNK / 2; w >= 1; w >>= 1) {
-      const bool upper = l & w;
+      const bool upper = l & mask;
 #pragma unroll
       for (int i = 0; i < w; ++i) {
         const float send = upper ? part[i] : part[i + w];
         const float keep = upper ? part[i + w] : part[i];
-        part[i] = keep + __shfl_xor_sync(0xffffffffu, send, w);
+        part[i] = keep + __shfl_xor_sync(0xffffffffu, send, mask);
       }
+      mask >>= 1;
     }
-    if (l < nt && col < P)
-      a.o[(size_t)(t0 + l) * a.heads * P + (size_t)head * P + col] = fmaf(bs[l], vs[l * TM_COLS + cb], part[0]);
+    if constexpr (LOG == 4) part[0] += __shfl_xor_sync(0xffffffffu, part[0], 1);
+    const int tok = l >> (LOG - 3);
+    if ((l & (LPC / 8 - 1)) == 0 && tok < nt && col < P)
+      a.o[(size_t)(t0 + tok) * a.heads * P + (size_t)head * P + col] = fmaf(bs[tok], vs[tok * COLS + cb], part[0]);
     if (next > 0) put(sm + (turn ^ 1) * PER);
     __syncthreads();
   }
 #pragma unroll
   for (int j = 0; j < RPL / 4; ++j) {
-    const int n = (8 * j + l) * 4;
+    const int n = (LPC * j + l) * 4;
     if (col < P && n < D) {
       if (a.vec) *reinterpret_cast<float4*>(st + n) = make_float4(S[4 * j], S[4 * j + 1], S[4 * j + 2], S[4 * j + 3]);
       else {
@@ -297,13 +295,14 @@ __global__ void __launch_bounds__(TM_THREADS) time_mixing_kernel(TimeMixArgs a) 
   }
 }
 
-template <typename AT, int RPL>
+template <typename AT, int RPL, int LPC>
 static int launch_time_mix(const TimeMixArgs& a, int S, cudaStream_t stream) {
-  const size_t smem = 2 * time_mix_buffer(RPL) * sizeof(float);
+  const size_t smem = 2 * time_mix_buffer(RPL, LPC) * sizeof(float);
   if (smem > 48 * 1024)
-    cudaFuncSetAttribute(time_mixing_kernel<AT, RPL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-  const dim3 grid((a.P + TM_COLS - 1) / TM_COLS, a.heads, S);
-  const cudaError_t e = launch_pdl(time_mixing_kernel<AT, RPL>, grid, dim3(TM_THREADS), smem, stream, a);
+    cudaFuncSetAttribute(time_mixing_kernel<AT, RPL, LPC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  const int cols = TM_THREADS / LPC;
+  const dim3 grid((a.P + cols - 1) / cols, a.heads, S);
+  const cudaError_t e = launch_pdl(time_mixing_kernel<AT, RPL, LPC>, grid, dim3(TM_THREADS), smem, stream, a);
   return e == cudaSuccess ? FT_OK : (int)e;
 }
 
@@ -351,10 +350,10 @@ int ft_time_mixing_scan(const void* r, const void* k, const void* v, long long l
   a.vec = !(D & 3) && !(slot_stride & 3) && !((uintptr_t)state & 15);
   int rc = FT_OK;
   FT_DISPATCH(dtype, AT, {
-    if (D <= 32) rc = launch_time_mix<AT, 4>(a, S, stream);
-    else if (D <= 64) rc = launch_time_mix<AT, 8>(a, S, stream);
-    else if (D <= 128) rc = launch_time_mix<AT, 16>(a, S, stream);
-    else rc = launch_time_mix<AT, 32>(a, S, stream);
+    if (D <= 32) rc = launch_time_mix<AT, 4, 8>(a, S, stream);
+    else if (D <= 64) rc = launch_time_mix<AT, 4, 16>(a, S, stream);
+    else if (D <= 128) rc = launch_time_mix<AT, 8, 16>(a, S, stream);
+    else rc = launch_time_mix<AT, 16, 16>(a, S, stream);
   });
   if (rc != FT_OK) return rc;
   FT_LAUNCH_CHECK();

@@ -72,7 +72,7 @@ def write_safetensors(path: str, tensors: Dict[str, torch.Tensor]) -> None:
     header, blobs, at = {}, [], 0
     for name, t in tensors.items():
         t = t.contiguous()
-        raw = t.view(torch.uint8).numpy().tobytes() if t.numel() else b""
+        raw = t.reshape(-1).view(torch.uint8).numpy().tobytes() if t.numel() else b""
         header[name] = {"dtype": _CODES[t.dtype], "shape": list(t.shape), "data_offsets": [at, at + len(raw)]}
         blobs.append(raw)
         at += len(raw)

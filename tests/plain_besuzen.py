@@ -110,11 +110,11 @@ def time_mixing_scan(r, k, v, w, u):
     return out
 
 
-def time_mixing(h, p, W, c, eps):
+def time_mixing(h, p, W, c, eps, store=lambda v: v):
     T = h.shape[0]
     H, D = c["heads"], c["dim"]
-    r, k, v, g = (shifted_mix(h, W[p + "mu." + n]) @ W[p + n].T for n in "rkvg")
-    low = torch.tanh(shifted_mix(h, W[p + "mu.w"]) @ W[p + "w1"].T)
+    r, k, v, g = (store(store(shifted_mix(h, W[p + "mu." + n])) @ W[p + n].T) for n in "rkvg")
+    low = torch.tanh(store(shifted_mix(h, W[p + "mu.w"])) @ W[p + "w1"].T)
     w = torch.exp(-torch.exp(low @ W[p + "w2"].T + W[p + "w0"]))
     o = time_mixing_scan(r.view(T, H, D), k.view(T, H, D), v.view(T, H, D), w.view(T, H, D), W[p + "u"])
     o = o / torch.sqrt((o * o).mean(-1, keepdim=True) + eps)
@@ -125,53 +125,126 @@ def glu(h, p, W, act):
     return (act(h @ W[p + "gate"].T) * (h @ W[p + "up"].T)) @ W[p + "down"].T
 
 
-def choose_experts(z, router):
-    """``(ids, weights)`` of one token from its router logits ``z``."""
+def choose_experts(z, router, ids=None):
+    """``(ids, weights, margin)`` of one token from its router logits ``z``: the best groups by their largest
+    score, the best experts inside them; ``margin``: how far (in score) the choice is from another one.
+    With ``ids`` those experts are taken instead."""
     s = torch.softmax(z, -1)
     E, top = router["experts"], router["top"]
     groups = router.get("groups") or {"count": 1, "keep": 1}
-    per = E // groups["count"]
-    best = sorted(range(groups["count"]), key=lambda g: (-float(s[g * per:(g + 1) * per].max()), g))[:groups["keep"]]
-    allowed = [e for g in best for e in range(g * per, (g + 1) * per)]
-    ids = sorted(allowed, key=lambda e: (-float(s[e]), e))[:top]
-    w = s[ids]
-    return ids, w / (w.sum() + 1e-20)
+    count, keep = groups["count"], groups["keep"]
+    per = E // count
+    value = [float(s[g * per:(g + 1) * per].max()) for g in range(count)]
+    order = sorted(range(count), key=lambda g: (-value[g], g))
+    allowed = [e for g in sorted(order[:keep]) for e in range(g * per, (g + 1) * per)]
+    ranked = sorted(allowed, key=lambda e: (-float(s[e]), e))
+    margin = float("inf")
+    if len(ranked) > top:
+        margin = float(s[ranked[top - 1]] - s[ranked[top]])
+    if keep < count:
+        margin = min(margin, value[order[keep - 1]] - value[order[keep]])
+    chosen = ranked[:top] if ids is None else [int(e) for e in ids]
+    w = s[chosen]
+    return chosen, w / (w.sum() + 1e-20), margin
 
 
-def routed(h, p, W, c):
+def routed(h, p, W, c, ids=None, margins=None):
     z = h @ W[p + "router"].T
     out = torch.zeros_like(h)
+    found = []
     for t in range(h.shape[0]):
-        ids, w = choose_experts(z[t], c["router"])
-        for e, we in zip(ids, w):
+        chosen, w, margin = choose_experts(z[t], c["router"], None if ids is None else ids[t])
+        found.append(margin)
+        for e, we in zip(chosen, w):
             out[t] += we * glu(h[t:t + 1], f"{p}e{e}.", W, silu)[0]
+    if margins is not None:
+        margins.append(torch.tensor(found))
     if c.get("shared"):
         out = out + torch.sigmoid(h @ W[p + "shared.sg"].T) * glu(h, p + "shared.", W, silu)
     return out
 
 
-def feed_forward(h, p, W, c):
-    return glu(h, p, W, gelu_tanh) if c["kind"] == "dense" else routed(h, p, W, c)
-
-
-def forward(tokens, W, config, layers_out=None):
-    """Logits ``[T, vocab]``; with a list in ``layers_out`` also the residual stream after every layer."""
+def forward(config, W, tokens, expert_ids=None, margins=None, layers_out=None, store=lambda v: v):
+    """Logits ``[T, vocab]``.  ``store`` is applied to what an engine with 16-bit activations stores (the sublayers'
+    inputs and outputs, a time mixer's mixes and projections): with a function that perturbs its argument by as
+    much as such a rounding, the result shows how far rounding alone moves each position.  ``expert_ids``: ``{layer: [T, top]}``, experts to take instead of the chosen ones;
+    ``margins`` (a list) takes every routed layer's margins ``[T]``, ``layers_out`` (a list) the residual stream
+    after every layer."""
     eps = config["norm"]["eps"]
-    x = W["embed"][tokens] * config["embedding"]["scale"]
+    x = W["embed"][torch.as_tensor(tokens)] * config["embedding"]["scale"]
     first = None
     for i, layer in enumerate(config["layers"]):
-        p, m = f"l{i}.", layer["mixer"]
-        h = layer_norm(x, W[p + "norm1"], eps)
+        p, m, mlp = f"l{i}.", layer["mixer"], layer.get("mlp")
+        h = store(layer_norm(x, W[p + "norm1"], eps))
         if layer["type"] == "attention":
             y, v = attention(h, p + "mix.", W, m, first)
             if m.get("v_mix") and first is None:
                 first = v
         else:
             y = (m["left_scale"] * head_gated_attention(h, p + "mix.left.", W, m["left"])
-                 + m["right_scale"] * time_mixing(h, p + "mix.right.", W, m["right"], eps))
-        if layer.get("mlp"):
-            y = y + feed_forward(layer_norm(x, W[p + "norm2"], eps), p + "mlp.", W, layer["mlp"])
+                 + m["right_scale"] * time_mixing(h, p + "mix.right.", W, m["right"], eps, store))
+        y = store(y)
+        if mlp:
+            g = store(layer_norm(x, W[p + "norm2"], eps))
+            if mlp["kind"] == "dense":
+                y = y + glu(g, p + "mlp.", W, gelu_tanh)
+            else:
+                y = y + routed(g, p + "mlp.", W, mlp, (expert_ids or {}).get(i), margins)
         x = x + y
         if layers_out is not None:
             layers_out.append(x.clone())
     return layer_norm(x, W["final.norm"], eps) @ W["head"].T * config["logit_scale"]
+
+
+def expected_tensors(config):
+    """Name -> shape of every tensor of a model of ``config`` (``mixer.right.low_rank`` filled in)."""
+    width = config["width"]
+    out = {"embed": (config["vocab"], width), "final.norm": (width,), "head": (config["vocab"], width)}
+
+    def linear(name, rows, cols, bias=False):
+        out[name] = (rows, cols)
+        if bias:
+            out[name + ".b"] = (rows,)
+
+    def gated(p, ff):
+        linear(p + "gate", ff, width)
+        linear(p + "up", ff, width)
+        linear(p + "down", width, ff)
+
+    for i, layer in enumerate(config["layers"]):
+        p, m, mlp = f"l{i}.", layer["mixer"], layer.get("mlp")
+        out[p + "norm1"] = (width,)
+        scopes = [("mix.", m)] if layer["type"] == "attention" else [("mix.left.", m["left"])]
+        for scope, a in scopes:
+            linear(p + scope + "q", a["heads"] * a["dim"], width, True)
+            linear(p + scope + "k", a["kv_heads"] * a["dim"], width, True)
+            linear(p + scope + "v", a["kv_heads"] * a["vdim"], width, True)
+            linear(p + scope + "g", a["heads"] * (a["vdim"] if scope == "mix." else 1), width)
+            linear(p + scope + "o", width, a["heads"] * a["vdim"])
+        if layer["type"] == "attention":
+            if m.get("v_mix"):
+                out[p + "mix.vmix"] = ()
+        else:
+            r = p + "mix.right."
+            n = m["right"]["heads"] * m["right"]["dim"]
+            for name in "rkvgw":
+                out[r + "mu." + name] = (width,)
+            for name in "rkvg":
+                linear(r + name, n, width)
+            linear(r + "w1", m["right"]["low_rank"], width)
+            linear(r + "w2", n, m["right"]["low_rank"])
+            out[r + "w0"] = out[r + "norm"] = (n,)
+            out[r + "u"] = (m["right"]["heads"], m["right"]["dim"])
+            linear(r + "o", width, n)
+        if mlp:
+            out[p + "norm2"] = (width,)
+            if mlp["kind"] == "dense":
+                gated(p + "mlp.", mlp["ff"])
+            else:
+                linear(p + "mlp.router", mlp["router"]["experts"], width)
+                for e in range(mlp["router"]["experts"]):
+                    gated(f"{p}mlp.e{e}.", mlp["expert"]["ff"])
+                if mlp.get("shared"):
+                    gated(p + "mlp.shared.", mlp["shared"]["ff"])
+                    linear(p + "mlp.shared.sg", 1, width)
+    return out
