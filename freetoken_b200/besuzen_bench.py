@@ -113,6 +113,13 @@ def kernel_pairs(s: Dict[str, int], peaks: Dict[str, Any], reps: int = 10) -> Di
             lambda i: ops.channel_delta_scan(qkv[i], beta, decay, w0, a_log, states[i], y, slot, q, H, H, D, D, 1e-6,
                                              D ** -0.5), len(qkv), nbytes=T * inner * (6 + 4 + 4) + 2 * S * state_b)
         del rkv, qkv, states
+        ys = rotate(lambda: torch.randn(T, inner, device=dev), T * inner * 8, most=8)
+        gate, gout = torch.randn(T, inner, device=dev, dtype=bf), torch.empty(T, inner, device=dev, dtype=bf)
+        for name, groups in ((f"a norm per head of {D}", H), ("one norm a row", 1)):
+            run(f"gated_norm ({name}), {label}",
+                lambda i, g=groups: ops.gated_norm(ys[i], gate, u, gout, g, 1e-6, False), len(ys),
+                nbytes=T * inner * (4 + 2 + 2))
+        del ys
         N = 128
         C = inner + 2 * N
         xs = rotate(lambda: torch.randn(T, C, device=dev, dtype=bf) * 0.5, T * C * 2 + S * inner * N * 4)

@@ -50,6 +50,7 @@ LIBRARIES: Dict[str, str] = {
     "attention_prefill_mha": "attention_prefill_mha.cu",
     "moe_gemm_tc": "moe_gemm_tc.cu",
     "recurrent": "recurrent.cu",
+    "gated_norm": "gated_norm.cu",
     "time_mixing": "time_mixing.cu",
 }
 HEADERS: List[str] = ["common.cuh", "mma_utils.cuh", "tcgen05.cuh", "status_codes.h", "sampling_static.h"]

@@ -812,7 +812,7 @@ def time_mixing_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: t
     """Per head, with ``w = exp(-exp(decay + w0))`` per key channel: ``o_t = (S + diag(u) k_t v_t^T)^T r_t``, then ``S
     <- diag(w_t) S + k_t v_t^T``.  ``r`` and ``k`` are ``[T, heads * key_dim]``, ``v`` ``[T, heads * head_dim]`` (one
     row stride), ``decay`` float32; the state of head h lies at ``h * head_dim * key_dim`` of its slot's row, ``[head_dim,
-    key_dim]``."""
+    key_dim]``.  Every segment brings at least one token; as many tokens as segments: one each, a kernel of its own."""
     for name, t in (("r", r), ("k", k), ("v", v)):
         _need(t, name, r.dtype, contiguous=False)
     for name, t in (("decay", decay), ("state", state)):
@@ -828,10 +828,10 @@ def time_mixing_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: t
         raise KernelError("time_mixing_scan: shapes do not match")
     if len({t.stride(0) for t in (r, k, v)}) != 1 or any(t.stride(1) != 1 for t in (r, k, v, decay)):
         raise KernelError("time_mixing_scan: r, k and v need one row stride and unit column strides")
-    f = _fn("time_mixing", "ft_time_mixing_scan", "p p p q p q p p p q p p p i i i i i")
+    f = _fn("time_mixing", "ft_time_mixing_scan", "p p p q p q p p p q p p p i i i i i i")
     _check(f(_ptr(r), _ptr(k), _ptr(v), r.stride(0), _ptr(decay), decay.stride(0), _ptr(w0), _ptr(u), _ptr(state),
              state.stride(0), _ptr(o), _ptr(seg_slot), _ptr(seg_q_start), heads, head_dim, key_dim,
-             seg_slot.numel(), code(r.dtype), _stream()), "time_mixing_scan")
+             seg_slot.numel(), T, code(r.dtype), _stream()), "time_mixing_scan")
 
 
 GATES = {"silu": 0, "sigmoid": 1}
@@ -850,7 +850,7 @@ def gated_norm(y: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, out: t
     if gate.shape != y.shape or out.shape != y.shape or gate.stride(1) != 1 or width % groups \
             or width % weight.numel() or gate_kind not in GATES:
         raise KernelError("gated_norm: shapes do not match")
-    f = _fn("recurrent", "ft_gated_norm", "p p q p i p i i i f i i i")
+    f = _fn("gated_norm", "ft_gated_norm", "p p q p i p i i i f i i i")
     _check(f(_ptr(y), _ptr(gate), gate.stride(0), _ptr(weight), weight.numel(), _ptr(out), T, width, groups,
              float(eps), int(gate_first), GATES[gate_kind], code(out.dtype), _stream()), "gated_norm")
 

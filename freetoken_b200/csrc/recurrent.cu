@@ -1,6 +1,6 @@
 // Mixers that carry a state of fixed size from token to token: a short causal
 // convolution over time, a selective state space with one decay per head
-// (Mamba-2's recurrence), the gated delta rule, and the gated norm behind both.
+// (Mamba-2's recurrence) and the gated delta rule (the gated norm behind them: gated_norm.cu).
 //
 // Everything that enters a recurrence is float32 whatever the activation type:
 // step sizes (softplus), decays (exp), gates (sigmoid), unit norms and the state
@@ -14,7 +14,6 @@
 //                    taps-1 inputs of a request live in its state slot
 //   ssd_scan         S <- exp(-exp(A) dt) S + dt B x^T ; y = S^T C + D x       (S: N x P per head)
 //   delta_scan       S <- g S ; u = beta (v - S^T k) ; S <- S + k u^T ; o = S^T q   (S: D x P per head)
-//   gated_norm       rms over groups of a row, a gate silu(z) before or after it
 //
 // State layout per head: [N or D][P] float32, P contiguous.  A warp owns WC
 // columns of a head's state and its lanes split the rows, so a column's dot
@@ -28,12 +27,6 @@ namespace ft {
 
 __device__ __forceinline__ float silu_f(float v) { return v / (1.f + expf(-v)); }
 __device__ __forceinline__ float softplus_f(float v) { return v > 20.f ? v : log1pf(expf(v)); }
-// a gate's function: 0 silu, 1 sigmoid
-__device__ __forceinline__ float gate_f(float v, int kind) {
-  const float sg = 1.f / (1.f + expf(-v));
-  return kind == 1 ? sg : v * sg;
-}
-
 // Sums V values per lane over the warp with V - 1 + log2(32 / V) shuffles: at every step a lane
 // hands half of its values to the lane `mask` away and adds what it gets to the half it keeps.
 // Afterwards v[0] of lane l is the warp's total of value  l >> (5 - log2 V).
@@ -693,104 +686,6 @@ __global__ void __launch_bounds__(SCAN_THREADS) delta_scan_kernel(DeltaArgs a) {
   }
 }
 
-// --------------------------------------------------------------------- gated norm
-// A row of `width` float32 values in `groups` equal parts, each divided by its own root mean
-// square; times weight[i % weight_len]; a gate silu(z) (or sigmoid(z)) on the values before the norm
-// (gate_first) or on the result.  One warp per (token, group).
-template <typename AT>
-__global__ void __launch_bounds__(128) gated_norm_kernel(const float* __restrict__ y, const AT* __restrict__ z,
-                                                         long long ldz, const float* __restrict__ weight,
-                                                         int weight_len, AT* __restrict__ out, int T, int width,
-                                                         int groups, float eps, int gate_first, int gate_kind) {
-  pdl_wait();
-  const int lane = threadIdx.x & 31;
-  const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-  if (item >= (long long)T * groups) return;
-  const int t = (int)(item / groups), grp = (int)(item % groups);
-  const int size = width / groups, base = grp * size;
-  const float* row = y + (size_t)t * width + base;
-  const AT* gate = z + (size_t)t * ldz + base;
-  float ss = 0.f;
-  for (int i = lane; i < size; i += 32) {
-    float v = row[i];
-    if (gate_first) v *= gate_f(to_float(gate[i]), gate_kind);
-    ss = fmaf(v, v, ss);
-  }
-  const float inv = 1.f / sqrtf(warp_sum(ss) / (float)size + eps);
-  AT* dst = out + (size_t)t * width + base;
-  for (int i = lane; i < size; i += 32) {
-    const float gv = gate_f(to_float(gate[i]), gate_kind);
-    float v = row[i];
-    if (gate_first) v *= gv;
-    v = v * inv * weight[(base + i) % weight_len];
-    if (!gate_first) v *= gv;
-    dst[i] = from_float<AT>(v);
-  }
-}
-
-// The same norm with TPI threads per (token, group), 16-byte pieces, and every value kept in
-// registers between the sum of squares and the scaling: parts of up to 4 * KEEP * TPI values, a
-// multiple of 4, rows 16-byte (bfloat16 gate: 8-byte) aligned.
-__device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ float4 ld4(const __nv_bfloat16* p) {
-  const uint2 raw = *reinterpret_cast<const uint2*>(p);
-  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
-  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
-  return make_float4(a.x, a.y, b.x, b.y);
-}
-__device__ __forceinline__ void st4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
-__device__ __forceinline__ void st4(__nv_bfloat16* p, float4 v) {
-  uint2 raw;
-  *reinterpret_cast<__nv_bfloat162*>(&raw.x) = __floats2bfloat162_rn(v.x, v.y);
-  *reinterpret_cast<__nv_bfloat162*>(&raw.y) = __floats2bfloat162_rn(v.z, v.w);
-  *reinterpret_cast<uint2*>(p) = raw;
-}
-
-template <typename AT, int TPI, int KEEP>
-__global__ void __launch_bounds__(128) gated_norm_vec_kernel(const float* __restrict__ y, const AT* __restrict__ z,
-                                                             long long ldz, const float* __restrict__ weight,
-                                                             int weight_len, AT* __restrict__ out, int T, int width,
-                                                             int groups, float eps, int gate_first, int gate_kind) {
-  __shared__ float scratch[33];
-  pdl_wait();
-  const int sub = threadIdx.x % TPI;
-  const long long item = (long long)blockIdx.x * (128 / TPI) + threadIdx.x / TPI;
-  if (item >= (long long)T * groups) return;          // a warp (TPI 32) or the whole block (TPI 128) leaves
-  const int t = (int)(item / groups), grp = (int)(item % groups);
-  const int size = width / groups, base = grp * size, pieces = size >> 2;
-  const float* row = y + (size_t)t * width + base;
-  const AT* gate = z + (size_t)t * ldz + base;
-  float4 keep[KEEP], gk[KEEP];
-  float ss = 0.f;
-#pragma unroll
-  for (int j = 0; j < KEEP; ++j) {
-    const int gi = sub + j * TPI;
-    if (gi < pieces) {
-      float4 v = ld4(row + 4 * gi);
-      const float4 gr = ld4(gate + 4 * gi);
-      const float4 gv = make_float4(gate_f(gr.x, gate_kind), gate_f(gr.y, gate_kind), gate_f(gr.z, gate_kind), gate_f(gr.w, gate_kind));
-      if (gate_first) { v.x *= gv.x; v.y *= gv.y; v.z *= gv.z; v.w *= gv.w; }
-      keep[j] = v;
-      gk[j] = gv;
-      ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss); ss = fmaf(v.z, v.z, ss); ss = fmaf(v.w, v.w, ss);
-    }
-  }
-  ss = TPI == 32 ? warp_sum(ss) : block_sum(ss, scratch);
-  const float inv = 1.f / sqrtf(ss / (float)size + eps);
-  AT* dst = out + (size_t)t * width + base;
-#pragma unroll
-  for (int j = 0; j < KEEP; ++j) {
-    const int gi = sub + j * TPI;
-    if (gi < pieces) {
-      const float4 w = ld4(weight + (base + 4 * gi) % weight_len);
-      float4 v = keep[j];
-      v.x *= inv * w.x; v.y *= inv * w.y; v.z *= inv * w.z; v.w *= inv * w.w;
-      if (!gate_first) { v.x *= gk[j].x; v.y *= gk[j].y; v.z *= gk[j].z; v.w *= gk[j].w; }
-      st4(dst + 4 * gi, v);
-    }
-  }
-}
-
 // A few segments of a long prompt leave most SMs without a block when a warp owns 8 columns:
 // then a warp owns 2 and four times as many blocks share the work.
 #ifndef NARROW_WC
@@ -939,43 +834,6 @@ int ft_retention_scan(const void* qkv, long long ld, const float* decay, const f
   DeltaArgs a{qkv, nullptr, nullptr, decay, nullptr, state, o, seg_slot, seg_q_start, ld, 0, slot_stride,
               heads, P, D, heads, 0.f, k_scale, 0, nullptr, 0, cos_sin, seg_pos0, cos_sin ? rot_dims : 0};
   return dispatch_delta<2>(a, S, dtype, stream);
-}
-
-int ft_gated_norm(const float* y, const void* z, long long ldz, const float* weight, int weight_len, void* out,
-                  int T, int width, int groups, float eps, int gate_first, int gate_kind, int dtype,
-                  cudaStream_t stream) {
-  if (T <= 0) return FT_OK;
-  if (width <= 0 || groups <= 0 || width % groups || weight_len <= 0) return FT_ERR_SHAPE;
-  const long long items = (long long)T * groups;
-  const int size = width / groups;
-  const bool vec = !(size & 3) && !(weight_len & 3) && !(ldz & 3) && !((uintptr_t)y & 15) && !((uintptr_t)z & 15) &&
-                   !((uintptr_t)weight & 15) && !((uintptr_t)out & 15);
-  if (vec && size <= 16 * 32) {
-    FT_DISPATCH(dtype, AT, launch_pdl(gated_norm_vec_kernel<AT, 32, 4>, dim3((unsigned)((items + 3) / 4)), dim3(128), 0, stream,
-                                      y, (const AT*)z, ldz, weight, weight_len, (AT*)out, T, width, groups, eps,
-                                      gate_first, gate_kind));
-    FT_LAUNCH_CHECK();
-    return FT_OK;
-  }
-  if (vec && size <= 16 * 128) {
-    FT_DISPATCH(dtype, AT, launch_pdl(gated_norm_vec_kernel<AT, 128, 4>, dim3((unsigned)items), dim3(128), 0, stream, y,
-                                      (const AT*)z, ldz, weight, weight_len, (AT*)out, T, width, groups, eps,
-                                      gate_first, gate_kind));
-    FT_LAUNCH_CHECK();
-    return FT_OK;
-  }
-  if (vec && size <= 64 * 128) {
-    FT_DISPATCH(dtype, AT, launch_pdl(gated_norm_vec_kernel<AT, 128, 16>, dim3((unsigned)items), dim3(128), 0, stream, y,
-                                      (const AT*)z, ldz, weight, weight_len, (AT*)out, T, width, groups, eps,
-                                      gate_first, gate_kind));
-    FT_LAUNCH_CHECK();
-    return FT_OK;
-  }
-  const unsigned blocks = (unsigned)((items + 3) / 4);
-  FT_DISPATCH(dtype, AT, launch_pdl(gated_norm_kernel<AT>, dim3(blocks), dim3(128), 0, stream, y, (const AT*)z, ldz,
-                                    weight, weight_len, (AT*)out, T, width, groups, eps, gate_first, gate_kind));
-  FT_LAUNCH_CHECK();
-  return FT_OK;
 }
 
 }  // extern "C"

@@ -333,8 +333,9 @@ __device__ __forceinline__ unsigned branch_slots(const BranchArgs& b, int t, flo
   back = warp_sum(lane < b.k && id >= b.experts ? w : 0.f);
   return __ballot_sync(0xffffffffu, lane < b.k && id < b.experts);
 }
-// columns 4g .. 4g + 3 of token t's branch (k <= 32), the rows' pieces fetched four at a time
-template <typename AT>
+// columns 4g .. 4g + 3 of token t's branch (k <= 32), the rows' pieces fetched four at a time (PAIRS: those of the
+// other sublayer two at a time; with many tokens the registers that takes cost more than it gains)
+template <typename AT, bool PAIRS = false>
 __device__ __forceinline__ float4 branch_at4(const BranchArgs& b, int t, int H, int gi, unsigned slots, float back) {
   const AT* rows = (const AT*)b.rows + (size_t)t * b.k * H + 4 * gi;
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -346,13 +347,21 @@ __device__ __forceinline__ float4 branch_at4(const BranchArgs& b, int t, int H, 
   }
   if (b.beside) {
     const AT* other = (const AT*)b.beside + (size_t)t * b.kb * H + 4 * gi;
-    for (int j0 = 0; j0 < b.kb; j0 += 2) {
-      const bool second = j0 + 1 < b.kb;
-      const float4 v0 = load4f(other + (size_t)j0 * H), v1 = second ? load4f(other + (size_t)(j0 + 1) * H) : zero;
-      const float s0 = b.beside_scale ? b.beside_scale[j0] : 1.f;
-      const float s1 = b.beside_scale && second ? b.beside_scale[j0 + 1] : 1.f;
-      y.x = fmaf(s0, v0.x, y.x); y.y = fmaf(s0, v0.y, y.y); y.z = fmaf(s0, v0.z, y.z); y.w = fmaf(s0, v0.w, y.w);
-      y.x = fmaf(s1, v1.x, y.x); y.y = fmaf(s1, v1.y, y.y); y.z = fmaf(s1, v1.z, y.z); y.w = fmaf(s1, v1.w, y.w);
+    constexpr int STEP = PAIRS ? 2 : 1;
+    for (int j0 = 0; j0 < b.kb; j0 += STEP) {
+      float4 v[STEP];
+      float s[STEP];
+#pragma unroll
+      for (int q = 0; q < STEP; ++q) {
+        const bool in = j0 + q < b.kb;
+        v[q] = in ? load4f(other + (size_t)(j0 + q) * H) : zero;
+        s[q] = in && b.beside_scale ? b.beside_scale[j0 + q] : 1.f;
+      }
+#pragma unroll
+      for (int q = 0; q < STEP; ++q) {
+        y.x = fmaf(s[q], v[q].x, y.x); y.y = fmaf(s[q], v[q].y, y.y);
+        y.z = fmaf(s[q], v[q].z, y.z); y.w = fmaf(s[q], v[q].w, y.w);
+      }
     }
   }
   if (back != 0.f) h = load4f((const AT*)b.source + (size_t)t * H + 4 * gi);
@@ -580,7 +589,7 @@ __global__ void __launch_bounds__(THREADS) join_layer_norm_kernel(JoinNormArgs a
       if (gi < groups) {
         x[j] = load4f(r + 4 * gi);
         if (a.b.rows) {
-          const float4 z = branch_at4<AT>(a.b, t, H, gi, slots, back);
+          const float4 z = branch_at4<AT, EAGER>(a.b, t, H, gi, slots, back);
           x[j].x += z.x; x[j].y += z.y; x[j].z += z.z; x[j].w += z.w;
           store4f(r + 4 * gi, x[j]);
         }

@@ -112,8 +112,8 @@ __global__ void __launch_bounds__(128) token_shift_kernel(ShiftArgs a) {
 // A column of a head's state is shared by LPC lanes; lane l holds rows (LPC j + l) 4 .. + 3 for j < RPL / 4, so
 // that the lanes read consecutive pieces of r, k, w (and of the state, which is kept value by value: [P][D]).  A
 // warp owns 32 / LPC columns, a block of 8 warps 256 / LPC.  Tokens come in chunks of 8: every warp fetches one
-// token of the NEXT chunk into registers while the block works through the current chunk in shared memory and puts
-// it into the other of two buffers afterwards: one barrier a chunk.  The decay's exponentials and the bonus
+// token of a later chunk into registers while the block works through the current chunk in shared memory and puts
+// the next one into the other of two buffers afterwards: one barrier a chunk.  The decay's exponentials and the bonus
 // u . (r k) are formed on the way into shared memory.  The read-out's partial sums of the 8 tokens are added over the
 // lanes together, each lane ending with the total of one token: 8 shuffles a chunk.
 constexpr int TM_WARPS = 8;
@@ -182,24 +182,28 @@ __global__ void __launch_bounds__(TM_THREADS) time_mixing_kernel(TimeMixArgs a) 
     u[e] = n < D ? a.u[(size_t)head * D + n] : 0.f;
   }
 
-  // this warp stages token `warp` of a chunk, the first TM_CHUNK * COLS threads one value of v each
-  AT pr[NE], pk[NE], pv;
-  float pd[NE];
+  // this warp stages token `warp` of a chunk, the first TM_CHUNK * COLS threads one value of v each; two chunks
+  // are on their way in registers, so that a load from device memory has a whole chunk's time and more
+  struct Staged {
+    AT r[NE], k[NE], v;
+    float d[NE];
+  } even, odd;
   const int vt = threadIdx.x / COLS, vc = threadIdx.x % COLS;
-  auto fetch = [&](int t0, int nt) {
+  auto fetch = [&](int t0, Staged& x) {
+    const int nt = min(TM_CHUNK, q1 - t0);             // may be 0 or less: nothing is read
     const size_t t = t0 + warp;
 #pragma unroll
     for (int e = 0; e < NE; ++e) {
       const int n = lane + 32 * e;
       const bool in = warp < nt && n < D;
-      pr[e] = in ? rp[t * a.ld + n] : from_float<AT>(0.f);
-      pk[e] = in ? kp[t * a.ld + n] : from_float<AT>(0.f);
-      pd[e] = in ? dp[t * a.ld_decay + n] : 0.f;
+      x.r[e] = in ? rp[t * a.ld + n] : from_float<AT>(0.f);
+      x.k[e] = in ? kp[t * a.ld + n] : from_float<AT>(0.f);
+      x.d[e] = in ? dp[t * a.ld_decay + n] : 0.f;
     }
     const int c = blockIdx.x * COLS + vc;
-    pv = (vt < nt && c < P) ? vp[(size_t)(t0 + vt) * a.ld + c] : from_float<AT>(0.f);
+    x.v = (vt < nt && c < P) ? vp[(size_t)(t0 + vt) * a.ld + c] : from_float<AT>(0.f);
   };
-  auto put = [&](float* buf) {
+  auto put = [&](float* buf, const Staged& x) {
     float* rs = buf;
     float* ks = rs + TM_CHUNK * DP;
     float* ws = ks + TM_CHUNK * DP;
@@ -209,57 +213,75 @@ __global__ void __launch_bounds__(TM_THREADS) time_mixing_kernel(TimeMixArgs a) 
 #pragma unroll
     for (int e = 0; e < NE; ++e) {
       const int n = lane + 32 * e;
-      const float rv = to_float(pr[e]), kv = to_float(pk[e]);
+      const float rv = to_float(x.r[e]), kv = to_float(x.k[e]);
       rs[warp * DP + n] = rv;
       ks[warp * DP + n] = kv;
-      ws[warp * DP + n] = expf(-expf(pd[e] + w0[e]));
+      ws[warp * DP + n] = expf(-expf(x.d[e] + w0[e]));
       bonus = fmaf(rv * kv, u[e], bonus);
     }
     bonus = warp_sum(bonus);
     if (lane == 0) bs[warp] = bonus;
-    if (vt < TM_CHUNK) vs[threadIdx.x] = to_float(pv);
+    if (vt < TM_CHUNK) vs[threadIdx.x] = to_float(x.v);
   };
 
-  fetch(q0, min(TM_CHUNK, q1 - q0));
-  put(sm);
-  __syncthreads();
-  int turn = 0;
-  for (int t0 = q0; t0 < q1; t0 += TM_CHUNK, turn ^= 1) {
+  struct Row {
+    float4 r[RPL / 4], k[RPL / 4], w[RPL / 4];
+    float v;
+  };
+  // one chunk: works through tokens t0 .. from buffer `turn`, puts the next chunk (`x`) into the other one and
+  // fetches the chunk two further on in its place
+  auto chunk = [&](int t0, int turn, Staged& x) {
     const int nt = min(TM_CHUNK, q1 - t0);
-    const int next = min(TM_CHUNK, q1 - t0 - TM_CHUNK);
-    if (next > 0) fetch(t0 + TM_CHUNK, next);
     const float* rs = sm + turn * PER;
     const float* ks = rs + TM_CHUNK * DP;
     const float* ws = ks + TM_CHUNK * DP;
     const float* vs = ws + TM_CHUNK * DP;
     const float* bs = vs + TM_CHUNK * COLS;
     float part[TM_CHUNK];
-    auto token = [&](int tt) {
-      const float v = vs[tt * COLS + cb];
-      float acc = 0.f;
+    auto load_row = [&](int tt, Row& row) {
+      row.v = vs[tt * COLS + cb];
 #pragma unroll
       for (int j = 0; j < RPL / 4; ++j) {
         const int n = tt * DP + (LPC * j + l) * 4;
-        const float4 r4 = *reinterpret_cast<const float4*>(rs + n);
-        const float4 k4 = *reinterpret_cast<const float4*>(ks + n);
-        const float4 w4 = *reinterpret_cast<const float4*>(ws + n);
-        acc = fmaf(S[4 * j], r4.x, acc);
-        acc = fmaf(S[4 * j + 1], r4.y, acc);
-        acc = fmaf(S[4 * j + 2], r4.z, acc);
-        acc = fmaf(S[4 * j + 3], r4.w, acc);
-        S[4 * j] = fmaf(w4.x, S[4 * j], k4.x * v);
-        S[4 * j + 1] = fmaf(w4.y, S[4 * j + 1], k4.y * v);
-        S[4 * j + 2] = fmaf(w4.z, S[4 * j + 2], k4.z * v);
-        S[4 * j + 3] = fmaf(w4.w, S[4 * j + 3], k4.w * v);
+        row.r[j] = *reinterpret_cast<const float4*>(rs + n);
+        row.k[j] = *reinterpret_cast<const float4*>(ks + n);
+        row.w[j] = *reinterpret_cast<const float4*>(ws + n);
+      }
+    };
+    auto token = [&](const Row& row) {
+      float acc = 0.f;
+#pragma unroll
+      for (int j = 0; j < RPL / 4; ++j) {
+        acc = fmaf(S[4 * j], row.r[j].x, acc);
+        acc = fmaf(S[4 * j + 1], row.r[j].y, acc);
+        acc = fmaf(S[4 * j + 2], row.r[j].z, acc);
+        acc = fmaf(S[4 * j + 3], row.r[j].w, acc);
+        S[4 * j] = fmaf(row.w[j].x, S[4 * j], row.k[j].x * row.v);
+        S[4 * j + 1] = fmaf(row.w[j].y, S[4 * j + 1], row.k[j].y * row.v);
+        S[4 * j + 2] = fmaf(row.w[j].z, S[4 * j + 2], row.k[j].z * row.v);
+        S[4 * j + 3] = fmaf(row.w[j].w, S[4 * j + 3], row.k[j].w * row.v);
       }
       return acc;
     };
     if (nt == TM_CHUNK) {
+      Row cur, ahead;                                  // the next token's row is on its way meanwhile
+      load_row(0, cur);
 #pragma unroll
-      for (int tt = 0; tt < TM_CHUNK; ++tt) part[tt] = token(tt);
+      for (int tt = 0; tt < TM_CHUNK; ++tt) {
+        if (tt + 1 < TM_CHUNK) load_row(tt + 1, ahead);
+        part[tt] = token(cur);
+        cur = ahead;
+      }
     } else {
 #pragma unroll
-      for (int tt = 0; tt < TM_CHUNK; ++tt) part[tt] = tt < nt ? token(tt) : 0.f;
+      for (int tt = 0; tt < TM_CHUNK; ++tt) {
+        part[tt] = 0.f;
+        if (tt < nt) {
+          Row cur;
+          load_row(tt, cur);
+          part[tt] = token(cur);
+        }
+      }
     }
     // lane l of a column's ends with the total of token l >> (LOG - 3)
     int mask = LPC / 2;
@@ -278,8 +300,21 @@ __global__ void __launch_bounds__(TM_THREADS) time_mixing_kernel(TimeMixArgs a) 
     const int tok = l >> (LOG - 3);
     if ((l & (LPC / 8 - 1)) == 0 && tok < nt && col < P)
       a.o[(size_t)(t0 + tok) * a.heads * P + (size_t)head * P + col] = fmaf(bs[tok], vs[tok * COLS + cb], part[0]);
-    if (next > 0) put(sm + (turn ^ 1) * PER);
+    if (t0 + TM_CHUNK < q1) {
+      put(sm + (turn ^ 1) * PER, x);
+      fetch(t0 + 3 * TM_CHUNK, x);
+    }
     __syncthreads();
+  };
+
+  fetch(q0, even);
+  fetch(q0 + TM_CHUNK, odd);
+  put(sm, even);
+  fetch(q0 + 2 * TM_CHUNK, even);
+  __syncthreads();
+  for (int t0 = q0; t0 < q1; t0 += 2 * TM_CHUNK) {
+    chunk(t0, 0, odd);
+    if (t0 + TM_CHUNK < q1) chunk(t0 + TM_CHUNK, 1, even);
   }
 #pragma unroll
   for (int j = 0; j < RPL / 4; ++j) {
@@ -293,6 +328,140 @@ __global__ void __launch_bounds__(TM_THREADS) time_mixing_kernel(TimeMixArgs a) 
       }
     }
   }
+}
+
+// Segments of one token each (a decode step): what it costs is reading and writing the states, so a lane holds
+// its rows of r, k and w in registers, made once, and streams CPL columns of the state, all loads in flight
+// together, without shared memory.  Sums run in the order of the kernel above: a token's result does not depend on
+// which of the two it took.
+template <typename AT, int RPL, int LPC, int CPL>
+__global__ void __launch_bounds__(128) time_mixing_step_kernel(TimeMixArgs a) {
+  constexpr int NE = LPC * RPL / 32, NJ = RPL / 4;
+  constexpr int CPW = 32 / LPC;
+  constexpr int LOG = LPC == 8 ? 3 : 4;
+  static_assert(CPL <= LPC, "a lane per column when they are added up");
+  pdl_wait();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, l = lane & (LPC - 1);
+  const int head = blockIdx.y, seg = blockIdx.z;
+  const int D = a.D, P = a.P;
+  const int col0 = (blockIdx.x * 4 + warp) * CPL * CPW + (lane >> LOG);       // columns col0 + c * CPW
+  if ((blockIdx.x * 4 + warp) * CPL * CPW >= P) return;                        // the whole warp leaves
+  const size_t t = a.seg_q_start[seg];
+  float* st = a.state + (size_t)a.seg_slot[seg] * a.slot_stride + (size_t)head * P * D;
+  const AT* rp = (const AT*)a.r + t * a.ld + (size_t)head * D;
+  const AT* kp = (const AT*)a.k + t * a.ld + (size_t)head * D;
+  const AT* vp = (const AT*)a.v + t * a.ld + (size_t)head * P;
+  const float* dp = a.decay + t * a.ld_decay + (size_t)head * D;
+  const float* w0 = a.w0 + (size_t)head * D;
+  const float* up = a.u + (size_t)head * D;
+
+  float4 S[CPL][NJ];
+#pragma unroll
+  for (int c = 0; c < CPL; ++c)
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+      const int col = col0 + c * CPW, n = (LPC * j + l) * 4;
+      S[c][j] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (col < P && n < D) {
+        const float* p = st + (size_t)col * D + n;
+        if (a.vec) S[c][j] = *reinterpret_cast<const float4*>(p);
+        else {
+          S[c][j].x = p[0];
+          if (n + 1 < D) S[c][j].y = p[1];
+          if (n + 2 < D) S[c][j].z = p[2];
+          if (n + 3 < D) S[c][j].w = p[3];
+        }
+      }
+    }
+  float v[CPL];
+#pragma unroll
+  for (int c = 0; c < CPL; ++c) v[c] = col0 + c * CPW < P ? to_float(vp[col0 + c * CPW]) : 0.f;
+  float bonus = 0.f;
+#pragma unroll
+  for (int e = 0; e < NE; ++e) {
+    const int n = lane + 32 * e;
+    if (n < D) bonus = fmaf(to_float(rp[n]) * to_float(kp[n]), up[n], bonus);
+  }
+  bonus = warp_sum(bonus);
+  float part[CPL];
+#pragma unroll
+  for (int c = 0; c < CPL; ++c) part[c] = 0.f;
+#pragma unroll
+  for (int j = 0; j < NJ; ++j) {
+    float r[4], k[4], w[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int n = (LPC * j + l) * 4 + i;
+      const bool in = n < D;
+      r[i] = in ? to_float(rp[n]) : 0.f;
+      k[i] = in ? to_float(kp[n]) : 0.f;
+      w[i] = in ? expf(-expf(dp[n] + w0[n])) : 0.f;
+    }
+#pragma unroll
+    for (int c = 0; c < CPL; ++c) {
+      float4& s = S[c][j];
+      part[c] = fmaf(s.x, r[0], part[c]);
+      part[c] = fmaf(s.y, r[1], part[c]);
+      part[c] = fmaf(s.z, r[2], part[c]);
+      part[c] = fmaf(s.w, r[3], part[c]);
+      s.x = fmaf(w[0], s.x, k[0] * v[c]);
+      s.y = fmaf(w[1], s.y, k[1] * v[c]);
+      s.z = fmaf(w[2], s.z, k[2] * v[c]);
+      s.w = fmaf(w[3], s.w, k[3] * v[c]);
+    }
+  }
+#pragma unroll
+  for (int c = 0; c < CPL; ++c)
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+      const int col = col0 + c * CPW, n = (LPC * j + l) * 4;
+      if (col < P && n < D) {
+        float* p = st + (size_t)col * D + n;
+        if (a.vec) *reinterpret_cast<float4*>(p) = S[c][j];
+        else {
+          p[0] = S[c][j].x;
+          if (n + 1 < D) p[1] = S[c][j].y;
+          if (n + 2 < D) p[2] = S[c][j].z;
+          if (n + 3 < D) p[3] = S[c][j].w;
+        }
+      }
+    }
+  // a column's lanes are added up; the lanes share the columns out among themselves on the way
+  int mask = LPC / 2, mine = 0;
+#pragma unroll
+  for (int w = CPL / 2; w >= 1; w >>= 1) {
+    const bool upper = l & mask;
+    if (upper) mine += w;
+#pragma unroll
+    for (int i = 0; i < w; ++i) {
+      const float send = upper ? part[i] : part[i + w];
+      const float keep = upper ? part[i + w] : part[i];
+      part[i] = keep + __shfl_xor_sync(0xffffffffu, send, mask);
+    }
+    mask >>= 1;
+  }
+  const int first = 2 * mask - 1;                      // lanes with the same columns differ in these bits
+  for (; mask >= 1; mask >>= 1) part[0] += __shfl_xor_sync(0xffffffffu, part[0], mask);
+  const int col = col0 + mine * CPW;
+  if ((l & first) == 0 && col < P) {
+    float vm = v[0];
+#pragma unroll
+    for (int c = 1; c < CPL; ++c) vm = mine == c ? v[c] : vm;
+    a.o[t * a.heads * P + (size_t)head * P + col] = fmaf(bonus, vm, part[0]);
+  }
+}
+
+template <typename AT, int RPL, int LPC>
+static int launch_time_mix_step(const TimeMixArgs& a, int S, cudaStream_t stream) {
+  constexpr int MANY = 32 / RPL, FEW = RPL == 4 ? 2 : 1;   // columns a lane: plenty of blocks, or a few
+  auto grid = [&](int cpl) { return dim3((a.P + 4 * cpl * (32 / LPC) - 1) / (4 * cpl * (32 / LPC)), a.heads, S); };
+  const dim3 many = grid(MANY);
+  cudaError_t e;
+  if ((long long)many.x * many.y * many.z >= 2 * 148)
+    e = launch_pdl(time_mixing_step_kernel<AT, RPL, LPC, MANY>, many, dim3(128), 0, stream, a);
+  else
+    e = launch_pdl(time_mixing_step_kernel<AT, RPL, LPC, FEW>, grid(FEW), dim3(128), 0, stream, a);
+  return e == cudaSuccess ? FT_OK : (int)e;
 }
 
 template <typename AT, int RPL, int LPC>
@@ -342,13 +511,24 @@ int ft_token_shift(const void* x, long long ldx, const float* mu, void* out, flo
 
 int ft_time_mixing_scan(const void* r, const void* k, const void* v, long long ld, const float* decay,
                         long long ld_decay, const float* w0, const float* u, float* state, long long slot_stride,
-                        float* o, const int* seg_slot, const int* seg_q_start, int heads, int P, int D, int S,
+                        float* o, const int* seg_slot, const int* seg_q_start, int heads, int P, int D, int S, int T,
                         int dtype, cudaStream_t stream) {
   if (S <= 0) return FT_OK;
   if (heads <= 0 || P <= 0 || D <= 0 || D > 256 || heads > 65535 || S > 65535) return FT_ERR_SHAPE;
   TimeMixArgs a{r, k, v, decay, w0, u, state, o, seg_slot, seg_q_start, ld, ld_decay, slot_stride, heads, P, D, 0};
   a.vec = !(D & 3) && !(slot_stride & 3) && !((uintptr_t)state & 15);
   int rc = FT_OK;
+  if (T == S) {                                        // one token a segment
+    FT_DISPATCH(dtype, AT, {
+      if (D <= 32) rc = launch_time_mix_step<AT, 4, 8>(a, S, stream);
+      else if (D <= 64) rc = launch_time_mix_step<AT, 4, 16>(a, S, stream);
+      else if (D <= 128) rc = launch_time_mix_step<AT, 8, 16>(a, S, stream);
+      else rc = launch_time_mix_step<AT, 16, 16>(a, S, stream);
+    });
+    if (rc != FT_OK) return rc;
+    FT_LAUNCH_CHECK();
+    return FT_OK;
+  }
   FT_DISPATCH(dtype, AT, {
     if (D <= 32) rc = launch_time_mix<AT, 4, 8>(a, S, stream);
     else if (D <= 64) rc = launch_time_mix<AT, 4, 16>(a, S, stream);

@@ -65,7 +65,7 @@ class _Recurrent(Mixer):
         return cache.state[:, :cut], cache.state[:, cut:]
 
     def libraries(self, dtype) -> List[str]:
-        return ["recurrent"] + linear.libraries(dtype)
+        return ["recurrent", "gated_norm"] + linear.libraries(dtype)
 
 
 @register_mixer("ssd")
@@ -401,7 +401,7 @@ class TimeMixing(Mixer):
         self.w["mu"] = self.w["mu"].view(len(self.MIXES), self.hidden)
 
     def libraries(self, dtype) -> List[str]:
-        return ["time_mixing", "recurrent", "rowwise"] + linear.libraries(dtype)
+        return ["time_mixing", "gated_norm", "rowwise"] + linear.libraries(dtype)
 
     def forward(self, ctx: StepContext, x: torch.Tensor, cache: CacheView, out=None) -> torch.Tensor:
         T, ws, w = x.shape[0], ctx.workspace, self.w
