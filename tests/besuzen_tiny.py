@@ -61,11 +61,11 @@ BZ_A: Dict = model(150, 44, 1e-5, [
     parallel((2, 2, 5, 9), (3, 20, 1), 0.5, 1.1),
 ], embedding_scale=1.7, logit_scale=0.6)
 
-# sizes the tensor-core attention kernels take, some filled up to them (48 to 64, 80 to 128), pages of 64
+# sizes the tensor-core attention kernels take, some filled up to them (40 and 56 to 64, 80 to 128), pages of 64
 BZ_B: Dict = model(320, 128, 2e-6, [
     attention(8, 2, 64, 64, 32, base=5000.0, mlp=moe(8, 2, 64, 4, 2, shared=96)),
     parallel((4, 2, 64, 80), (4, 32, 16), 0.6, 0.8, dense(256)),
-    attention(4, 2, 48, 64, 48, base=500000.0, mlp=moe(6, 1, 48, 6, 3, shared=64)),
+    attention(6, 2, 56, 64, 40, base=500000.0, mlp=moe(6, 1, 48, 6, 3, shared=64)),
     attention(2, 2, 32, 64, 16, v_mix=False, base=30000.0),
     parallel((6, 6, 32, 32), (2, 64, 24), 1.0, 1.0, moe(16, 4, 32, 2, 1)),
     attention(8, 2, 40, 64, 24, base=1000.0, mlp=dense(192)),

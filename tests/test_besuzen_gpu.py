@@ -445,7 +445,7 @@ FAR = {
 
 @pytest.mark.parametrize("dtype", list(DTYPES))
 @pytest.mark.parametrize("kind", list(FAR))
-@pytest.mark.parametrize("dim,vdim,page", [(20, 12, 8), (32, 32, 16), (48, 64, 64), (128, 64, 64)])
+@pytest.mark.parametrize("dim,vdim,page", [(20, 12, 8), (32, 32, 16), (40, 64, 64), (128, 64, 64)])
 def test_a_far_key_decides(tmp_path, kind, dim, vdim, page, dtype):
     """The asking token finds its target at the very first position and right before, on and right after page
     borders, hundreds of keys back, from inside a prompt portion and as a decoded token."""
@@ -527,8 +527,8 @@ def test_the_previous_token_crosses_every_cut(tmp_path, dtype):
 # ------------------------------------------------- long prompts at sizes between tiny and real
 LONG = bz.model(640, 256, 1e-5, [
     bz.attention(8, 2, 64, 64, 32, base=1e5, mlp=bz.dense(512)),
-    bz.parallel((4, 2, 64, 128), (4, 64, 32), 0.8, 0.6, bz.moe(16, 4, 64, 4, 2, shared=128)),
-    bz.attention(4, 2, 48, 64, 48, base=1e6, mlp=bz.moe(8, 2, 96, 2, 1)),
+    bz.parallel((4, 4, 64, 112), (4, 64, 24), 0.9, 0.6, bz.moe(16, 4, 64, 4, 2, shared=128)),
+    bz.attention(6, 2, 56, 64, 40, base=2e6, mlp=bz.moe(8, 2, 96, 2, 1)),
 ], embedding_scale=0.9, logit_scale=0.7)
 
 
